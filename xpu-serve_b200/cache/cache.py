@@ -3,14 +3,17 @@
 Layer calls are grouped by what they need (parts/base.py: KVNeed, StateNeed). Calls
 that keep every key of the same geometry form one group with one page pool and one
 page table; calls that keep a window form another, whose pages behind the window are
-given back as a sequence grows; calls with a fixed-size state (the short convolution's
+given back as a sequence grows (but for the pages of a sequence's first positions, where the
+window keeps those); calls with a fixed-size state (the short convolution's
 last kernel-1 inputs here, any recurrent state elsewhere) form groups that hold one
 row per slot. Each group owns its storage. A slot's length is advanced only by
 `end_step`, and `begin_step` changes nothing unless everything the step needs is
 available (the reference leaves a failed step's state as it was,
 src/backend/cpu_ref/cpu_backend.cpp:157-177).
 
-Storage of a key/value call: [pages, planes (keys, values; one for a latent), kv_heads, page_size, head_dim].
+Storage of a key/value call: [pages, planes (keys, values; one for a latent), kv_heads, page_size, head_dim]; where values
+have another size than keys, [pages, kv_heads * page_size * (head_dim + v_dim)], a page being its keys [kv_heads, page_size,
+head_dim] and then its values [kv_heads, page_size, v_dim] (the same layout when the sizes are equal).
 Storage of a state call:     [max_slots, *shape].
 """
 from __future__ import annotations
@@ -44,14 +47,16 @@ class KVGroup:
         self.max_seq_pages = max_seq_pages
         # logical page -> physical page, -1 where none is held
         self.table = np.full((max_slots, max_seq_pages), -1, dtype=np.int32)
-        self.first_held = np.zeros(max_slots, dtype=np.int64)    # pages below it were given back
+        self.first_held = np.zeros(max_slots, dtype=np.int64)    # pages below it were given back, but for the first `kept`
+        self.kept = _ceil_div(need.keep_first, page_size) if need.window > 0 else 0
         self.end_held = np.zeros(max_slots, dtype=np.int64)      # pages from it on are not held yet
         self.version = 0      # grows whenever a row of `table` changes (a staged copy of the table is then stale)
         # one page more than the pool hands out: padding rows of a fixed-size batch write there
         self.dummy_page = n_pages
+        shape = ((need.planes, need.kv_heads, page_size, need.head_dim) if need.v_dim in (0, need.head_dim) or need.planes == 1
+                 else (need.kv_heads * page_size * (need.head_dim + need.v_dim),))
         self.storage: Dict[Tuple[int, int], torch.Tensor] = {
-            c: torch.zeros((n_pages + 1, need.planes, need.kv_heads, page_size, need.head_dim),
-                           dtype=dtype, device=device) for c in calls}
+            c: torch.zeros((n_pages + 1, *shape), dtype=dtype, device=device) for c in calls}
 
     def _first_needed_page(self, start: int) -> int:
         """The lowest page a query at position `start` or later can still see."""
@@ -75,7 +80,7 @@ class KVGroup:
 
     def trim(self, slot: int, length: int) -> None:
         first = min(self._first_needed_page(length), int(self.end_held[slot]))
-        lo = int(self.first_held[slot])
+        lo = max(int(self.first_held[slot]), self.kept)
         if first > lo:
             self.pages.give_back(int(p) for p in self.table[slot, lo:first])
             self.table[slot, lo:first] = -1
@@ -95,6 +100,8 @@ class KVGroup:
 
     def release(self, slot: int) -> None:
         lo, hi = int(self.first_held[slot]), int(self.end_held[slot])
+        if lo > 0 and self.kept > 0:
+            self.pages.give_back(int(p) for p in self.table[slot, :min(self.kept, lo)])
         self.pages.give_back(int(p) for p in self.table[slot, lo:hi])
         self.table[slot, :] = -1
         self.first_held[slot] = 0

@@ -5,8 +5,9 @@ from .saralix import SaralixConfig
 from .nimelorn import NimelornConfig
 from .tozarax import TozaraxConfig
 from .vekuzen import VekuzenConfig
+from .gararax import GararaxConfig
 from .spec import (AttentionSpec, LayerCall, LayerSpec, ModelSpec, NormSpec, RopeSpec,
                    ShortConvSpec, SwiGLUSpec)
 
-__all__ = ["ConfigError", "read_json", "Lfm3Config", "Lfm3Rope", "SaralixConfig", "NimelornConfig", "TozaraxConfig", "VekuzenConfig", "AttentionSpec", "LayerCall",
+__all__ = ["ConfigError", "read_json", "Lfm3Config", "Lfm3Rope", "SaralixConfig", "NimelornConfig", "TozaraxConfig", "VekuzenConfig", "GararaxConfig", "AttentionSpec", "LayerCall",
            "LayerSpec", "ModelSpec", "NormSpec", "RopeSpec", "ShortConvSpec", "SwiGLUSpec"]

@@ -43,7 +43,7 @@ class AttentionSpec:
     head_dim: int
     qk_norm: bool            # RMSNorm over head_dim on q and k, before the position encoding
     qk_norm_eps: float
-    position: Optional[RopeSpec]
+    position: Optional[object]   # a RopeSpec or a ScaledRopeSpec
     window: int              # 0: every earlier key is visible; W > 0: keys with pos - j < W
     head_gate: bool          # o[t, h, :] *= sigmoid((x Wg^T)[t, h])
     scale: float             # multiplies q.k before the softmax
@@ -52,13 +52,22 @@ class AttentionSpec:
         "v": "self_attn.v_proj.weight", "o": "self_attn.o_proj.weight",
         "gate": "self_attn.gate_proj.weight",
         "q_norm": "self_attn.q_norm.weight", "k_norm": "self_attn.k_norm.weight",
-        "q_bias": "self_attn.q_proj.bias", "k_bias": "self_attn.k_proj.bias", "v_bias": "self_attn.v_proj.bias"})
+        "q_bias": "self_attn.q_proj.bias", "k_bias": "self_attn.k_proj.bias", "v_bias": "self_attn.v_proj.bias",
+        "temp": "self_attn.temp"})
     kind: str = "attention"
     qkv_bias: bool = False   # q, k and v projections with a bias each (LFM3 has none)
-    v_dim: int = 0           # size of a value head when it differs from head_dim (0: head_dim); needs position None
+    v_dim: int = 0           # size of a value head when it differs from head_dim (0: head_dim); needs position None, or v_layout "own"
     chunk: int = 0           # C > 0: a query at pos sees the earlier keys of its own block only, j >= pos - pos % C
                              # (blocks of C positions counted from the sequence's position 0); excludes `window`
     own_kv: bool = True      # False: the layer has no k, v and k-norm tensors; its call reads another call's cache
+    v_layout: str = "padded"  # "padded": key and value heads share one padded size in the kernels and the cache; "own": each
+                             # has its own (a rotation may then stand beside value heads of another size)
+    keep_first: int = 0      # beside `window`: the sequence's first positions j < keep_first stay visible for good
+    unit_qk: bool = False    # q and k divided by their root mean square over head_dim (qk_norm_eps), behind the rotation, no weight
+    shared_kv: bool = False  # the values are the keys as projected (no v tensors, one vector a position in the cache)
+    plus_one: bool = False   # softmax weights exp(s_j) / (1 + sum exp(s_j))
+    out_gate: bool = False   # every channel of the concatenated heads times sigmoid((x Wg^T)[t, c]) (names["gate"])
+    head_temp: bool = False  # scores of head h times a learned number (names["temp"])
 
 
 @dataclass(frozen=True)
@@ -101,16 +110,29 @@ class RopeScalingSpec:
 
 
 @dataclass(frozen=True)
+class BandRopeScalingSpec:
+    """Rotation frequencies stretched by bands of wavelength l = 2 pi / f (as Llama 3.1 does): f stays where l < original /
+    high, becomes f / factor where l > original / low, and (1 - s) f / factor + s f with s = (original / l - low) /
+    (high - low) between the two. cos and sin stay as they are."""
+    factor: float
+    low: float
+    high: float
+    original: float
+
+
+@dataclass(frozen=True)
 class ScaledRopeSpec:
-    """A rotate-half rotation of the first `dims` channels of a vector of `head_dim` channels: pair i couples
-    channels i and i + dims/2 (not i + head_dim/2) and turns by pos * theta^(-2i/dims), scaled as `scaling` says
-    (None: as is). The table it gives has head_dim/2 entries a position when dims == head_dim, which the kernels
-    that know one pairing read; the mixers that use it ask for dims == head_dim."""
+    """A rotation of the first `dims` channels of a vector of `head_dim` channels: pair i couples channels i and
+    i + dims/2 (not i + head_dim/2), or with `pairing` "interleaved" channels 2i and 2i + 1, and turns by
+    pos * theta^(-2i/dims), scaled as `scaling` says (a RopeScalingSpec or a BandRopeScalingSpec; None: as is). The table
+    has head_dim/2 entries a position, the identity behind the first dims/2. The kernels know one pairing, i and
+    i + head_dim/2 of the vector they are given: a mixer whose checkpoint pairs otherwise reorders its weights' rows."""
     head_dim: int
     theta: float
     dims: int
-    scaling: Optional[RopeScalingSpec] = None
+    scaling: Optional[object] = None
     kind: str = "rope_scaled"
+    pairing: str = "half"
 
 
 @dataclass(frozen=True)
@@ -217,6 +239,18 @@ class SquaredReluSpec:
 
 
 @dataclass(frozen=True)
+class PolyNormSpec:
+    """down(act(up x)) with act(z) = a N(z) + b N(z^2) + c N(z^3) + e: powers element by element, N a division by the root
+    mean square over the token's `intermediate` values (`eps` inside the root), (a, b, c, e) four learned numbers
+    (names["act"])."""
+    hidden: int
+    intermediate: int
+    eps: float
+    names: Dict[str, str] = field(default_factory=lambda: {"up": "mlp.up", "down": "mlp.down", "act": "mlp.act"})
+    kind: str = "poly_norm"
+
+
+@dataclass(frozen=True)
 class ClampedGLUSpec:
     """down(g * sigmoid(alpha g) * (u + up_shift)) with g = min(gate x, limit), u = clamp(up x, -limit, limit)."""
     hidden: int
@@ -243,9 +277,11 @@ class RoutedExpertsSpec:
     sum only with `renorm`. `activation` "relu_squared": an expert is down(max(up x, 0)^2), without a gate matrix.
 
     `score` "softmax_all": a token's scores are the softmax over all router outputs; the experts are chosen by score plus
-    `correction` (when set) and weighted by their scores times `route_scale`, as they are. `identity` n > 0: the router has n
-    more outputs behind the experts'; such a choice stands for the token's input itself (times its weight) and has no
-    tensors. `shared` may be any gated unit's spec (ClampedGLUSpec, or SwiGLUSpec for a plain gated unit)."""
+    `correction` (when set) and weighted by their scores times `route_scale`, as they are, or with `renorm` divided by their
+    sum + `renorm_eps`. `identity` n > 0: the router has n more outputs behind the experts'; such a choice stands for the
+    token's input itself (times its weight) and has no tensors; `groups` then are groups of all outputs, experts and these
+    together. `shared` may be any gated unit's spec (ClampedGLUSpec, or SwiGLUSpec for a plain gated unit); without
+    `shared_gated` its output joins the sum as it is (no one-row matrix)."""
     hidden: int
     intermediate: int
     experts: int
@@ -266,6 +302,8 @@ class RoutedExpertsSpec:
     keep_groups: int = 1
     group_top: int = 2
     renorm: bool = False
+    renorm_eps: float = 0.0
+    shared_gated: bool = True
     activation: str = "gated"        # "gated" (SwiGLU, or the clamped unit with `limit`) | "relu_squared"
 
 
@@ -324,6 +362,7 @@ class NormSpec:
     eps: float
     kind: str = "rmsnorm"    # "layernorm": (x - mean) * (variance + eps)^(-1/2) * w, no bias (parts/layernorm.py)
     offset: float = 0.0      # rmsnorm: the stored weight stands around zero and the norm multiplies by offset + w
+    scale: float = 1.0       # rmsnorm: the norm's result times a constant (a branch's factor on its way into the stream)
 
 
 @dataclass(frozen=True)
@@ -347,7 +386,7 @@ class PairHashEmbeddingSpec:
 class TokenSideSpec:
     """A per-layer input from the token itself, behind the layer's last sublayer: with e = table[tok, offset : offset + dim]
     (a second token table that all layers share, `table` its name at the model's top level, `columns` wide),
-    h += unit_rms(P (gelu_tanh(G h) * e)) * w, the norm's weight plain (names "gate": [dim, width], "proj": [width, dim],
+    h += scale * unit_rms(P (gelu_tanh(G h) * e)) * w, the norm's weight plain (names "gate": [dim, width], "proj": [width, dim],
     "norm": [width], under the layer's prefix)."""
     dim: int
     offset: int
@@ -356,6 +395,7 @@ class TokenSideSpec:
     eps: float
     table: str = "side.embed"
     names: Dict[str, str] = field(default_factory=lambda: {"gate": "side.gate", "proj": "side.proj", "norm": "side.norm"})
+    scale: float = 1.0
 
 
 @dataclass(frozen=True)
@@ -382,6 +422,7 @@ class LayerSpec:
     depth_terms: int = 0     # n > 0: what the layer hands on is sum_j c[j] X_j over the embedding's output X_0 and the
                              # results X_1 .. X_(n-1) of the layers so far, this one's last (names "depth": [n])
     token_side: Optional[TokenSideSpec] = None   # "pre_norm": a gated slice of a second token table joins the stream last
+    branch_scale: float = 1.0   # sandwich layers: h += branch_scale * post(...) for both sublayers
 
 
 @dataclass(frozen=True)
@@ -394,6 +435,9 @@ class LayerCall:
     cache_of: Optional[int] = None
     mix_in: bool = False     # before this call the stream becomes M [stream; embedding output] (ModelSpec.names["pass_in"]:
                              # [width, 2 width]): how a pass over repeated layers starts
+    step_row: Optional[int] = None  # before this call row `step_row` of ModelSpec.names["pass_step"] ([pass_steps, width]) is
+                             # added to the stream: another way for a pass to start
+    add_embedding: bool = False  # ... and (first) the embedding output
 
 
 @dataclass(frozen=True)
@@ -413,14 +457,19 @@ class ModelSpec:
     prefixes: Tuple[str, ...] = ("model.",)   # tried in turn for "<prefix>embed_tokens.weight"
     ignorable: Tuple[str, ...] = ()           # regular expressions: tensors of a folder that match are neither needed nor refused
     embedding: Optional[object] = None        # a spec with a `kind` (registry.register_embedding); None: table[tok] * embed_scale
+    pass_steps: int = 0                       # rows of names["pass_step"] (0: the model has none)
     depth_history: bool = False               # the step keeps every layer's result (layers with `depth_terms` read them)
     names: Dict[str, str] = field(default_factory=lambda: {
         "embed": "embed_tokens.weight", "final_norm": "embedding_norm.weight",
-        "head": "lm_head.weight", "pass_in": "loop.in"})   # "head" is looked up without the model prefix
+        "head": "lm_head.weight", "pass_in": "loop.in", "pass_step": "loop.step"})   # "head" is looked up without the model prefix
 
     @property
     def mixes_in(self) -> bool:
         return any(c.mix_in for c in self.order)
+
+    @property
+    def adds_embedding(self) -> bool:
+        return any(c.add_embedding for c in self.order)
 
     def shared_tables(self) -> Dict[str, Tuple[int, int]]:
         """Tensors at the model's top level that the layers read (name -> shape): the token-side tables."""
@@ -444,6 +493,8 @@ class ModelSpec:
         for i, call in enumerate(self.order):
             if not 0 <= call.layer < len(self.layers):
                 raise ValueError(f"order[{i}] names layer {call.layer} of {len(self.layers)}")
+            if call.step_row is not None and not 0 <= call.step_row < self.pass_steps:
+                raise ValueError(f"order[{i}] adds row {call.step_row} of {self.pass_steps} pass vectors")
             if call.cache_of is not None:
                 if not 0 <= call.cache_of < i:
                     raise ValueError(f"order[{i}] reads the cache of call {call.cache_of}, which does not run before it")

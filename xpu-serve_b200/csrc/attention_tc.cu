@@ -19,7 +19,8 @@
 //
 // S of block j + 1 is issued before P V of block j, so the tensor pipe works while the softmax of block j
 // runs. Every mbarrier wait is bounded (see tc_common.cuh); a CTA that gives up frees its tensor memory and
-// sets *status. Head size 64, groups that divide 128, one key split; other cases take the mma.sync kernel.
+// sets *status. A window may keep the sequence's first positions visible: their blocks are walked before the window's; a cache
+// with one plane holds keys that are the values too. Head size 64, groups that divide 128, one key split; other cases take the mma.sync kernel.
 // The reference's counterpart is its XMX flash kernel for prefill (src/backend/sycl/sycl_flash_attention.cpp:1-15).
 #include <cuda.h>
 
@@ -45,6 +46,10 @@ struct AttnTcParams {
     __nv_bfloat16* out;              // [T, Hq, D]
     int* status;
     int Hq, Hkv, G, tokens_per_tile, window;
+    int keep;                        // beside a window: the sequence's first positions that stay visible
+    int planes;                      // 1: the keys are the values too: loaded once, read by both products
+    int plus_one;                    // the softmax's denominator has one more term of score 0
+    int gate_channels;               // gate logits per channel instead of per head
     float scale_log2;
     int order;
 };
@@ -147,9 +152,10 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap tmap_kv, const AttnTcPar
     const int nt = min(p.tokens_per_tile, q_len - t0);
     const int kv_len = p.kv_lens[seq];
     const int pos0 = kv_len - q_len + t0;
-    const int hi = pos0 + nt;                                  // keys [lo, hi) matter to this tile
-    const int lo = xs_first_visible(pos0, p.window);
-    const int b_lo = lo / TN, nb = (hi + TN - 1) / TN - b_lo;
+    const int hi = pos0 + nt;                                  // keys from hi on do not matter to this tile
+    const XsBlocks blocks = xs_blocks(pos0, hi, p.window, p.keep, TN);
+    const int nb = blocks.count;
+    const bool own_v = p.planes > 1;
     const int32_t* table = p.page_table + (int64_t)seq * p.P;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int G = p.G;
@@ -207,22 +213,22 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap tmap_kv, const AttnTcPar
             int page[2], valid[2];                             // physical page (-1: none), rows of it inside the sequence
 #pragma unroll
             for (int h = 0; h < 2; ++h) {
-                const int lp = 2 * (b_lo + j) + h;
+                const int lp = 2 * blocks.at(j) + h;
                 const int rows = min(PAGE, kv_len - lp * PAGE);
                 page[h] = (rows > 0 && lp < p.P) ? table[lp] : -1;
                 valid[h] = page[h] >= 0 ? rows : 0;
             }
             const bool fix = valid[0] < PAGE || valid[1] < PAGE;
-            const uint32_t bytes = (uint32_t)((page[0] >= 0) + (page[1] >= 0)) * 2u * kPageBytes;
+            const uint32_t bytes = (uint32_t)((page[0] >= 0) + (page[1] >= 0)) * (own_v ? 2u : 1u) * kPageBytes;
             const uint32_t bar = smem_u32(fix ? &bar_fix[s] : &bar_kv_full[s]);
             if (lane == 0) {
                 if (bytes > 0) mbar_expect_tx(bar, bytes); else mbar_arrive_cta(bar);
 #pragma unroll
                 for (int h = 0; h < 2; ++h) {
                     if (page[h] < 0) continue;
-                    const int y = ((page[h] * 2 + 0) * p.Hkv + kvh) * PAGE;
+                    const int y = (page[h] * p.planes * p.Hkv + kvh) * PAGE;
                     tma_load_2d(smem_u32(stage + h * kPageBytes), &tmap_kv, 0, y, bar);
-                    tma_load_2d(smem_u32(stage + 2 * kPageBytes + h * kPageBytes), &tmap_kv, 0, y + p.Hkv * PAGE, bar);
+                    if (own_v) tma_load_2d(smem_u32(stage + 2 * kPageBytes + h * kPageBytes), &tmap_kv, 0, y + p.Hkv * PAGE, bar);
                 }
             }
             if (fix) {
@@ -231,7 +237,7 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap tmap_kv, const AttnTcPar
                 ++fixes[s];
 #pragma unroll
                 for (int h = 0; h < 2; ++h) {
-                    uint8_t* v_page = stage + 2 * kPageBytes + h * kPageBytes;
+                    uint8_t* v_page = stage + (own_v ? 2 * kPageBytes : 0) + h * kPageBytes;
                     for (int i = valid[h] * 8 + lane; i < PAGE * 8; i += 32)      // 16-byte chunks from row valid[h] on
                         *reinterpret_cast<uint4*>(v_page + i * 16) = make_uint4(0, 0, 0, 0);
                 }
@@ -266,7 +272,7 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap tmap_kv, const AttnTcPar
         if (lane == 0) {
             constexpr uint32_t idesc_o = instr_desc_mn(TM, D, true);
             const uint64_t dp0 = smem_desc_sw128(smem_u32(p_sm));
-            const uint64_t dv0 = smem_desc_sw128_mn(smem_u32(kv_sm + 2 * kPageBytes));
+            const uint64_t dv0 = smem_desc_sw128_mn(smem_u32(kv_sm + (own_v ? 2 * kPageBytes : 0)));
             for (int j = 0; j < nb && !*abort_p; ++j) {
                 const int s = j % KV_STAGES, buf = j & 1;
                 if (!mbar_wait(smem_u32(&bar_kv_full[s]), (j / KV_STAGES) & 1, abort_p)) break;
@@ -305,9 +311,9 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap tmap_kv, const AttnTcPar
         for (int j = grp; j < nb; j += 2, ++done) {
             if (!mbar_wait(smem_u32(&bar_s_full[grp]), done & 1, abort_p)) { bad = true; break; }
             tcgen05_fence_after();
-            const int key0 = (b_lo + j) * TN;
+            const int key0 = blocks.at(j) * TN;
             // a block that every row of the tile sees whole needs no test per key
-            const bool plain = pos >= 0 && key0 + TN - 1 <= pos0 && key0 >= xs_first_visible(pos0 + nt - 1, p.window);
+            const bool plain = pos >= 0 && key0 + TN - 1 <= pos0 && (key0 >= xs_first_visible(pos0 + nt - 1, p.window) || key0 + TN <= p.keep);
             // this row's 128 scores of the block, read once and kept through both passes
             uint32_t raw[TN];
 #pragma unroll
@@ -321,7 +327,7 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap tmap_kv, const AttnTcPar
 #pragma unroll
                 for (int e = 0; e < TN; ++e) {
                     const int key = key0 + e;
-                    const bool see = key <= pos && key >= lo_row;      // pos -1: nothing
+                    const bool see = key <= pos && (key >= lo_row || key < p.keep);      // pos -1: nothing
                     if (!see) raw[e] = 0xff800000u;                // -inf: its weight will be exactly 0
                     mx4[e & 3] = fmaxf(mx4[e & 3], __uint_as_float(raw[e]));
                 }
@@ -409,9 +415,10 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap tmap_kv, const AttnTcPar
             const float mb = mm == -INFINITY ? 0.0f : mm;
             const float a0 = ex2(m - mb), a1 = ex2(m1 - mb);
             l = l * a0 + l1 * a1;
+            if (p.plus_one) l += exp2f(-mm);
             const int t = tok_begin + t0 + r / G, h = kvh * G + r % G;
             float f = l > 0.0f ? 1.0f / l : 0.0f;
-            if (p.gate != nullptr) f *= 1.0f / (1.0f + __expf(-__bfloat162float(p.gate[(int64_t)t * p.ld_gate + h])));
+            if (p.gate != nullptr && !p.gate_channels) f *= 1.0f / (1.0f + __expf(-__bfloat162float(p.gate[(int64_t)t * p.ld_gate + h])));
             const float f0 = a0 * f, f1 = a1 * f;
             uint4* dst = reinterpret_cast<uint4*>(p.out + ((int64_t)t * p.Hq + h) * D);
 #pragma unroll
@@ -419,6 +426,16 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap tmap_kv, const AttnTcPar
                 float v[8];
 #pragma unroll
                 for (int e = 0; e < 8; ++e) v[e] = o[8 * c + e] * f0 + merge[(8 * c + e) * TM + r] * f1;
+                if (p.gate_channels) {
+                    const uint4 graw = *reinterpret_cast<const uint4*>(p.gate + (int64_t)t * p.ld_gate + h * D + 8 * c);
+                    const __nv_bfloat162* g2 = reinterpret_cast<const __nv_bfloat162*>(&graw);
+#pragma unroll
+                    for (int e = 0; e < 4; ++e) {
+                        const float2 z = __bfloat1622float2(g2[e]);
+                        v[2 * e] *= 1.0f / (1.0f + __expf(-z.x));
+                        v[2 * e + 1] *= 1.0f / (1.0f + __expf(-z.y));
+                    }
+                }
                 dst[c] = make_uint4(pack_bf16(v[0], v[1]), pack_bf16(v[2], v[3]), pack_bf16(v[4], v[5]), pack_bf16(v[6], v[7]));
             }
         }
@@ -443,8 +460,9 @@ XS_API int xs_attention_tc_supports(int D, int page_size, int G) {
 // max_kv_len: the longest sequence's keys, or 0 if the host does not know; it only picks the order in which CTAs start.
 XS_API int xs_attention_tc(const void* q, const void* pool, int64_t pool_pages, const int32_t* page_table, int P,
                            const int32_t* cu_seqlens, const int32_t* kv_lens, const void* gate, int64_t ld_gate, void* out,
-                           int T, int n_seqs, int max_q_len, int Hq, int Hkv, int D, int page_size, float scale, int window,
-                           int max_kv_len, int* status, cudaStream_t stream) {
+                           int T, int n_seqs, int max_q_len, int Hq, int Hkv, int D, int planes, int page_size, float scale,
+                           int window, int keep, int plus_one, int gate_channels, int max_kv_len, int* status,
+                           cudaStream_t stream) {
     if (T == 0) return 0;
     XS_REQUIRE(Hq > 0 && Hkv > 0 && Hq % Hkv == 0, "attention: %d heads over %d kv heads", Hq, Hkv);
     const int G = Hq / Hkv;
@@ -455,8 +473,11 @@ XS_API int xs_attention_tc(const void* q, const void* pool, int64_t pool_pages, 
     XS_REQUIRE(n_seqs <= 65535 && Hkv <= 65535, "attention (tcgen05): grid too large");
     XS_REQUIRE((uintptr_t)q % 16 == 0 && (uintptr_t)pool % 16 == 0 && (uintptr_t)out % 16 == 0,
                "attention (tcgen05): operands must be 16-byte aligned");
+    XS_REQUIRE((planes == 1 || planes == 2) && keep >= 0 && scale > 0.0f, "attention (tcgen05): %d planes, %d kept, scale %g", planes, keep, (double)scale);
+    XS_REQUIRE(gate == nullptr || !gate_channels || (ld_gate % 8 == 0 && (uintptr_t)gate % 16 == 0),
+               "attention (tcgen05): a gate per channel needs 16-byte rows");
     alignas(64) CUtensorMap map;
-    XS_REQUIRE(make_map(&map, pool, pool_pages * 2 * Hkv * PAGE, D, D, PAGE), "attention (tcgen05): the cache's tensor map could not be made");
+    XS_REQUIRE(make_map(&map, pool, pool_pages * planes * Hkv * PAGE, D, D, PAGE), "attention (tcgen05): the cache's tensor map could not be made");
     AttnTcParams p;
     p.q = (const __nv_bfloat16*)q;
     p.page_table = page_table;
@@ -472,6 +493,10 @@ XS_API int xs_attention_tc(const void* q, const void* pool, int64_t pool_pages, 
     p.G = G;
     p.tokens_per_tile = TM / G;
     p.window = window;
+    p.keep = window > 0 ? keep : 0;
+    p.planes = planes;
+    p.plus_one = plus_one;
+    p.gate_channels = gate != nullptr ? gate_channels : 0;
     p.scale_log2 = scale * 1.4426950408889634f;
     // All kv heads of the latest tiles first (5 to 15 % faster up to 8,192 keys: the long tiles of every head start
     // before any short one) while the keys and values of all heads together stay well inside L2; one head after the

@@ -91,6 +91,21 @@ __device__ __forceinline__ bool xs_visible(int pos, int key, int window) {
     return key <= pos && key >= xs_first_visible(pos, window);
 }
 
+// The blocks of `bn` keys that queries from position pos0 on can see, for a mask whose first `keep` positions stay visible
+// beside a sliding window: the kept blocks that lie before the window's first block, then the window's own. i counts the
+// blocks to walk, at(i) names the i-th.
+struct XsBlocks {
+    int kept, first, count;
+    __device__ __forceinline__ int at(int i) const { return i < kept ? i : first + (i - kept); }
+};
+__device__ __forceinline__ XsBlocks xs_blocks(int pos0, int hi, int window, int keep, int bn) {
+    XsBlocks b;
+    b.first = xs_first_visible(pos0, window) / bn;
+    b.kept = min((keep + bn - 1) / bn, b.first);
+    b.count = b.kept + (hi + bn - 1) / bn - b.first;
+    return b;
+}
+
 static inline int ceil_div_i(int64_t a, int64_t b) { return (int)((a + b - 1) / b); }
 
 // ---- programmatic dependent launch ------------------------------------------------------------

@@ -232,13 +232,15 @@ __global__ void moe_route_warp_kernel(const float* __restrict__ logits, int ld, 
 // correction (a number per expert). The experts form `groups` equal groups of neighbours; a group's score is the sum of its
 // `group_top` largest choice scores, and only experts of the `keep` best groups can be chosen (the others count as minus
 // infinity, so negative choice scores still beat them). The `top` largest choice scores are chosen (ties: the lower index,
-// for groups and for experts); the weights are the chosen experts' s times `scale`, not normed to sum 1 unless `renorm`.
+// for groups and for experts); the weights are the chosen experts' s times `scale`, divided by their sum + `renorm_eps` only
+// with `renorm`.
 // `score` 1: s is the softmax over all E logits instead of their sigmoids. Experts from `real` on have no weights (their
 // output is their input): a choice of one is written as id -1, with its weight.
 // A warp per token; the token's s and c stand in shared memory (2 E floats a warp).
 __global__ void moe_route_grouped_kernel(const float* __restrict__ logits, int ld, int T, int E, int top,
                                          const float* __restrict__ correction, int groups, int keep, int group_top, float scale,
-                                         int renorm, int score, int real, int32_t* __restrict__ ids, float* __restrict__ wts) {
+                                         int renorm, float renorm_eps, int score, int real, int32_t* __restrict__ ids,
+                                         float* __restrict__ wts) {
     extern __shared__ float route_smem[];
     pdl_launch_dependents();
     pdl_wait();
@@ -331,7 +333,7 @@ __global__ void moe_route_grouped_kernel(const float* __restrict__ logits, int l
     }
     if (lane < top) {
         ids[(int64_t)t * top + lane] = mine_id < real ? mine_id : -1;        // (an expert without weights: its input passes)
-        wts[(int64_t)t * top + lane] = (renorm ? mine / sum : mine) * scale;
+        wts[(int64_t)t * top + lane] = (renorm ? mine / (sum + renorm_eps) : mine) * scale;
     }
 }
 
@@ -587,8 +589,8 @@ XS_API int xs_moe_route(const float* logits, int ld, int T, int E, int top, floa
 }
 
 XS_API int xs_moe_route_grouped(const float* logits, int ld, int T, int E, int top, const float* correction, int groups, int keep,
-                                int group_top, float scale, int renorm, int score, int real, int32_t* ids, float* wts,
-                                cudaStream_t stream) {
+                                int group_top, float scale, int renorm, float renorm_eps, int score, int real, int32_t* ids,
+                                float* wts, cudaStream_t stream) {
     if (T == 0) return 0;
     XS_REQUIRE(T > 0 && E > 0 && top > 0 && top <= E && top <= kMaxTop && ld >= E,
                "moe_route_grouped: %d tokens, %d experts (row stride %d), top %d (at most %d)", T, E, ld, top, kMaxTop);
@@ -601,7 +603,7 @@ XS_API int xs_moe_route_grouped(const float* logits, int ld, int T, int E, int t
     XS_REQUIRE(per_warp <= 40 * 1024, "moe_route_grouped: %d experts are more than the kernel's shared memory holds", E);
     const int warps = per_warp * 4 <= 40 * 1024 ? 4 : 1;
     xs_launch(moe_route_grouped_kernel, dim3(ceil_div_i(T, warps)), dim3(32 * warps), per_warp * warps, stream, logits, ld, T, E, top,
-              correction, groups, keep, group_top, scale, renorm, score, real, ids, wts);
+              correction, groups, keep, group_top, scale, renorm, renorm_eps, score, real, ids, wts);
     XS_LAUNCH_CHECK("moe_route_grouped");
     return 0;
 }

@@ -413,6 +413,35 @@ __global__ void cast_rows_vec_kernel(const float* __restrict__ src, int64_t lds,
     }
 }
 
+// How a pass over repeated layers starts: the embedding's output (base) and the pass's own vector (row) join the stream.
+__global__ void stream_add_kernel(float* __restrict__ h, const float* __restrict__ base, const float* __restrict__ row, int64_t total, int n) {
+    pdl_launch_dependents();
+    pdl_wait();
+    for (int64_t i = (int64_t)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += (int64_t)gridDim.x * blockDim.x) {
+        float v = h[i];
+        if (base != nullptr) v += base[i];
+        if (row != nullptr) v += row[i % n];
+        h[i] = v;
+    }
+}
+
+__global__ void stream_add_vec_kernel(float4* __restrict__ h, const float4* __restrict__ base, const float4* __restrict__ row, int64_t total, int n4) {
+    pdl_launch_dependents();
+    pdl_wait();
+    for (int64_t i = (int64_t)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += (int64_t)gridDim.x * blockDim.x) {
+        float4 v = h[i];
+        if (base != nullptr) {
+            const float4 b = base[i];
+            v.x += b.x; v.y += b.y; v.z += b.z; v.w += b.w;
+        }
+        if (row != nullptr) {
+            const float4 r = row[i % n4];
+            v.x += r.x; v.y += r.y; v.z += r.z; v.w += r.w;
+        }
+        h[i] = v;
+    }
+}
+
 }  // namespace
 
 XS_API int xs_embed_pos(const void* table, const void* rows, int dtype, const int32_t* ids, const int32_t* positions, float* h,
@@ -538,6 +567,21 @@ XS_API int xs_causal_conv(const void* x, int64_t ldx, const float* taps_w, void*
                                     (TT*)state, cu_seqlens, slots, C, taps));
         XS_LAUNCH_CHECK("causal_conv (state)");
     }
+    return 0;
+}
+
+// h[t, :] += base[t, :] (when given) + row[:] (when given), all float32, n a row's width.
+XS_API int xs_stream_add(float* h, const float* base, const float* row, int T, int n, cudaStream_t stream) {
+    if (T == 0) return 0;
+    XS_REQUIRE(T > 0 && n > 0 && (base != nullptr || row != nullptr), "stream_add: %d rows of %d", T, n);
+    const bool vec = n % 4 == 0 && (uintptr_t)h % 16 == 0 && (uintptr_t)base % 16 == 0 && (uintptr_t)row % 16 == 0;
+    const int64_t total = (int64_t)T * n / (vec ? 4 : 1);
+    const int blocks = (int)((total + 255) / 256 < 148 * 16 ? (total + 255) / 256 : 148 * 16);
+    if (vec)
+        xs_launch(stream_add_vec_kernel, dim3(blocks), dim3(256), 0, stream, (float4*)h, (const float4*)base, (const float4*)row, total, n / 4);
+    else
+        xs_launch(stream_add_kernel, dim3(blocks), dim3(256), 0, stream, h, base, row, total, n);
+    XS_LAUNCH_CHECK("stream_add");
     return 0;
 }
 

@@ -94,6 +94,8 @@ class Model:
         tables = {SHARED + name: weights[name] for name in spec.shared_tables()}
         # the matrix that mixes the stream with the embedding's output in front of a pass over repeated layers
         self.pass_in = rt.matrix(weights[spec.names["pass_in"]]) if spec.mixes_in else None
+        # vectors that passes over repeated layers start with, one per pass
+        self.pass_step = rt.vector(weights[spec.names["pass_step"]]) if spec.pass_steps else None
         for layer in spec.layers:
             own = {k[len(layer.prefix):]: v for k, v in weights.items() if k.startswith(layer.prefix)}
             own.update(tables)
@@ -392,9 +394,18 @@ class Model:
             # front of every pass, and one product with the mixing matrix gives the pass's stream (float32)
             pair = rt.ws.get("pass_pair", (ctx.n_tokens, 2 * spec.hidden), rt.act_dtype)
             ops.cast_rows(h, pair[:, spec.hidden:])
+        embedded = None
+        if spec.adds_embedding:
+            embedded = rt.ws.get("embedded", (ctx.n_tokens, spec.hidden), torch.float32)
+            embedded.copy_(h)
         last = len(spec.order) - 1
         passes = 0
         for i, call in enumerate(spec.order):
+            if call.add_embedding or call.step_row is not None:
+                stream.flush(self.final_norm)
+                stream.changed()
+                ops.stream_add(stream.h, embedded if call.add_embedding else None,
+                               self.pass_step[call.step_row] if call.step_row is not None else None)
             if call.mix_in:
                 stream.flush(self.final_norm)
                 ops.cast_rows(stream.h, pair[:, :spec.hidden])
@@ -402,7 +413,9 @@ class Model:
                 stream.replace(rt.linear(pair, self.pass_in, f"stream_pass{passes & 1}", out_dtype=torch.float32))
             # the norm that reads the stream after this block, for products that carry the norm with them (none across a
             # mix, which rewrites the stream)
-            next_norm = self.final_norm if i == last else None if spec.order[i + 1].mix_in else self.blocks[spec.order[i + 1].layer].first_norm
+            nxt = spec.order[i + 1] if i < last else None
+            rewritten = nxt is not None and (nxt.mix_in or nxt.add_embedding or nxt.step_row is not None)
+            next_norm = self.final_norm if nxt is None else None if rewritten else self.blocks[nxt.layer].first_norm
             self.blocks[call.layer].forward(stream, ctx, cache.views[i], next_norm)
         if ctx.want_rows.numel() == 0:
             stream.flush(self.final_norm)

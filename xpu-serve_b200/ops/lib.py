@@ -44,17 +44,17 @@ def _signatures(lib) -> None:
         "xs_lightning_scan": [P, L, I, I, I, P, P, P, P, P, I, I, I, I, I, P, P, I, P, P],
         "xs_zero_rows": [P, P, I, L, P],
         "xs_gemm_generic": [P, P, P, P, I, I, I, I, I, L, L, L, P],
-        "xs_qk_norm_rope_store": [P, L, P, P, P, I, P, P, P, P, P, I, I, I, I, I, F, I, I, P],
-        "xs_attention_generic": [P, P, P, I, P, P, P, L, P, I, I, I, I, I, F, I, I, P],
+        "xs_qk_norm_rope_store": [P, L, P, P, P, I, P, P, P, P, P, I, I, I, I, I, I, P, I, F, I, I, P],
+        "xs_attention_generic": [P, P, P, I, P, P, P, L, P, I, I, I, I, I, I, I, F, I, I, I, I, I, P],
         "xs_short_conv": [P, L, P, P, P, P, P, P, P, I, I, I, I, I, I, P],
         "xs_attention_mma": [P, P, P, I, P, P, P, L, P, P, L, I, I, I, I, I, I, I, F, I, I, P],
-        "xs_attention_tc": [P, P, L, P, I, P, P, P, L, P, I, I, I, I, I, I, I, F, I, I, P, P],
+        "xs_attention_tc": [P, P, L, P, I, P, P, P, L, P, I, I, I, I, I, I, I, I, F, I, I, I, I, I, P, P],
         "xs_gemm_small_m": [P, P, P, P, P, I, I, I, I, L, L, L, I, I, P, L, P],
         "xs_gemm_small_m_normed": [P, P, P, P, P, I, I, I, I, L, L, L, I, I, P, L, P, I, I, F, P, P, L, P, P],
         "xs_gemm_small_m_ex": [P, P, P, P, P, I, I, I, I, L, L, L, I, I, P, L, P, I, I, F, P, P, L, P,
                                P, P, P, P, P, P, I, I, P, P, P, P],
         "xs_gemm_small_m_rope": [P, P, P, P, I, I, I, L, L, L, P, I, I, F, P, P, P, I, P, P, P, P, P, I, I, I, I, F, P],
-        "xs_attention_mma_merged": [P, P, P, I, P, P, P, L, P, P, L, P, L, P, I, I, I, I, I, I, I, F, I, I, P],
+        "xs_attention_mma_merged": [P, P, P, I, P, P, P, L, P, P, L, P, L, P, I, I, I, I, I, I, I, I, I, F, I, I, I, I, I, P],
         "xs_gemm_tc": [P, P, P, P, I, I, I, I, I, L, L, L, I, P, L, P, P],
         "xs_argmax": [P, L, I, I, P, P, P],
         "xs_sample": [P, L, I, I, P, P, P, P, P, P, I, P, P],
@@ -86,7 +86,9 @@ def _signatures(lib) -> None:
         "xs_depth_average": [P, L, P, I, P, L, P],
         "xs_rmsnorm_accumulate": [P, I, P, P, I, I, F, F, I, P],
         "xs_gated_delta_scan": [P, L, I, I, I, P, L, P, P, P, P, P, P, I, I, I, I, I, F, F, I, I, P],
-        "xs_moe_route_grouped": [P, I, I, I, I, P, I, I, I, F, I, I, I, P, P, P],
+        "xs_moe_route_grouped": [P, I, I, I, I, P, I, I, I, F, I, F, I, I, P, P, P],
+        "xs_poly_norm": [P, L, P, P, I, I, F, I, P],
+        "xs_stream_add": [P, P, P, I, I, P],
         "xs_mamba2_scan": [P, P, L, I, P, P, P, P, P, P, P, I, I, I, I, I, I, P],
         "xs_mamba2_scan_chunked": [P, P, L, I, P, P, P, P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, P],
     }
@@ -102,11 +104,11 @@ def _signatures(lib) -> None:
     lib.xs_attention_mma_scratch_bytes.restype = c_int64
     lib.xs_attention_mma_scratch_bytes.argtypes = [c_int64, c_int, c_int]
     lib.xs_attention_mma_supports.restype = c_int
-    lib.xs_attention_mma_supports.argtypes = [c_int, c_int, c_int]
+    lib.xs_attention_mma_supports.argtypes = [c_int, c_int, c_int, c_int]
     lib.xs_attention_tc_supports.restype = c_int
     lib.xs_attention_tc_supports.argtypes = [c_int, c_int, c_int]
     lib.xs_attention_mma_decode_slots.restype = c_int
-    lib.xs_attention_mma_decode_slots.argtypes = [c_int, c_int64]
+    lib.xs_attention_mma_decode_slots.argtypes = [c_int, c_int, c_int64]
     lib.xs_gemm_small_m_supports.restype = c_int
     lib.xs_gemm_small_m_supports.argtypes = [c_int, c_int, c_int64, c_int64]
     lib.xs_gemm_tc_supports.restype = c_int
@@ -384,26 +386,58 @@ def gemm_generic(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, bias: Opti
                                   M, N, K, x.stride(0), w.stride(0), out.stride(0), _stream()))
 
 
+def kv_page_shape(kv_heads: int, page_size: int, head_dim: int, v_dim: int, planes: int) -> tuple:
+    """The shape of one page of a key/value cache (cache/cache.py)."""
+    if planes == 2 and v_dim != head_dim:
+        return (kv_heads * page_size * (head_dim + v_dim),)
+    return (planes, kv_heads, page_size, head_dim)
+
+
+def _need_pool(pool: torch.Tensor, kv_heads: int, page_size: int, head_dim: int, v_dim: int, planes: int, dtype) -> None:
+    _need(pool, "cache", dtype)
+    shape = kv_page_shape(kv_heads, page_size, head_dim, v_dim, planes)
+    if tuple(pool.shape[1:]) != shape or (planes == 1 and v_dim != head_dim):
+        raise KernelError(f"cache is {tuple(pool.shape)}, expected [*, {', '.join(str(n) for n in shape)}]")
+
+
+def _need_gate(gate: Optional[torch.Tensor], q: torch.Tensor, heads: int, v_dim: int, channels: bool) -> int:
+    """The gate's row stride (0 without one)."""
+    if gate is None:
+        return 0
+    T, columns = q.shape[0], heads * v_dim if channels else heads
+    if gate.dtype != q.dtype or gate.stride(1) != 1 or gate.shape[0] != T or gate.shape[1] < columns:
+        raise KernelError(f"gate is {tuple(gate.shape)} {gate.dtype} for {T} tokens of {columns} gates")
+    return gate.stride(0)
+
+
 def qk_norm_rope_store(qkv: torch.Tensor, q_out: torch.Tensor, pool: Optional[torch.Tensor],
                        page_table: Optional[torch.Tensor], seq_of_token: torch.Tensor, positions: torch.Tensor,
                        q_w: Optional[torch.Tensor], k_w: Optional[torch.Tensor], rope: Optional[torch.Tensor],
-                       heads: int, kv_heads: int, head_dim: int, page_size: int, eps: float, write_kv: bool) -> None:
+                       heads: int, kv_heads: int, head_dim: int, page_size: int, eps: float, write_kv: bool,
+                       v_dim: int = 0, planes: int = 2, q_scale: Optional[torch.Tensor] = None) -> None:
+    """Columns [q heads | k heads | v heads] of qkv: per-head norms and rotation of q (to q_out, times `q_scale` [heads] when
+    given) and k, and keys and values into the cache's pages. `v_dim` (0: head_dim) is a value head's size; planes 1: there
+    are no values."""
+    v_dim = v_dim or head_dim
     _need(q_out, "q_out", qkv.dtype)
     if qkv.stride(1) != 1:
         raise KernelError("qkv rows must be contiguous")
     T = qkv.shape[0]
-    width = (heads + (2 * kv_heads if write_kv else 0)) * head_dim
+    width = heads * head_dim + (kv_heads * (head_dim + (v_dim if planes == 2 else 0)) if write_kv else 0)
     if qkv.shape[1] < width:
         raise KernelError(f"qkv is {tuple(qkv.shape)}, needs {width} columns")
     if write_kv:
-        _need(pool, "cache", qkv.dtype); _need(page_table, "page table", torch.int32)
-        if tuple(pool.shape[1:]) != (2, kv_heads, page_size, head_dim):
-            raise KernelError(f"cache is {tuple(pool.shape)}, expected [*, 2, {kv_heads}, {page_size}, {head_dim}]")
+        _need_pool(pool, kv_heads, page_size, head_dim, v_dim, planes, qkv.dtype)
+        _need(page_table, "page table", torch.int32)
     for v, name in ((q_w, "q_norm"), (k_w, "k_norm")):
         if v is not None:
             _need(v, name, torch.float32)
             if v.numel() != head_dim:
                 raise KernelError(f"{name} has {v.numel()} elements for heads of {head_dim}")
+    if q_scale is not None:
+        _need(q_scale, "q_scale", torch.float32)
+        if q_scale.numel() != heads:
+            raise KernelError(f"q_scale has {q_scale.numel()} elements for {heads} heads")
     if rope is not None:
         _need(rope, "rope table", torch.float32)
         if tuple(rope.shape[1:]) != (head_dim // 2, 2):
@@ -411,39 +445,41 @@ def qk_norm_rope_store(qkv: torch.Tensor, q_out: torch.Tensor, pool: Optional[to
     P = 0 if page_table is None else page_table.shape[1]
     _check(load().xs_qk_norm_rope_store(
         qkv.data_ptr(), qkv.stride(0), q_out.data_ptr(), _ptr(pool), _ptr(page_table), P, seq_of_token.data_ptr(),
-        positions.data_ptr(), _ptr(q_w), _ptr(k_w), _ptr(rope), T, heads, kv_heads, head_dim, page_size, float(eps),
-        1 if write_kv else 0, _code(qkv), _stream()))
+        positions.data_ptr(), _ptr(q_w), _ptr(k_w), _ptr(rope), T, heads, kv_heads, head_dim, v_dim, int(planes), _ptr(q_scale),
+        page_size, float(eps), 1 if write_kv else 0, _code(qkv), _stream()))
 
 
 def attention_generic(q: torch.Tensor, pool: torch.Tensor, page_table: torch.Tensor, seq_of_token: torch.Tensor,
                       positions: torch.Tensor, gate: Optional[torch.Tensor], out: torch.Tensor, kv_heads: int,
-                      page_size: int, scale: float, window: int) -> None:
-    _need(q, "q"); _need(out, "out", q.dtype); _need(pool, "cache", q.dtype); _need(page_table, "page table", torch.int32)
+                      page_size: int, scale: float, window: int, keep: int = 0, planes: int = 2, plus_one: bool = False,
+                      gate_channels: bool = False) -> None:
+    """Attention over the paged cache, any even head size up to 256 (values: out's last dimension). `window` 0: every
+    earlier key; W > 0: keys with pos - j < W or j < keep; -C: the query's own block of C positions. planes 1: the keys are
+    the values. plus_one: the softmax's denominator has one more term of score 0. gate: logits per head, or with
+    gate_channels per channel."""
+    _need(q, "q"); _need(out, "out", q.dtype); _need(page_table, "page table", torch.int32)
     T, heads, D = q.shape
-    if tuple(pool.shape[1:]) != (2, kv_heads, page_size, D):
-        raise KernelError(f"cache is {tuple(pool.shape)}, expected [*, 2, {kv_heads}, {page_size}, {D}]")
-    ld_gate = 0
-    if gate is not None:
-        if gate.dtype != q.dtype or gate.stride(1) != 1 or gate.shape[0] != T or gate.shape[1] < heads:
-            raise KernelError(f"gate is {tuple(gate.shape)} {gate.dtype} for {T} tokens of {heads} heads")
-        ld_gate = gate.stride(0)
+    DV = out.shape[2]
+    _need_pool(pool, kv_heads, page_size, D, DV, planes, q.dtype)
+    ld_gate = _need_gate(gate, q, heads, DV, gate_channels)
     _check(load().xs_attention_generic(
         q.data_ptr(), pool.data_ptr(), page_table.data_ptr(), page_table.shape[1], seq_of_token.data_ptr(),
-        positions.data_ptr(), _ptr(gate), ld_gate, out.data_ptr(), T, heads, kv_heads, D, page_size, float(scale),
-        int(window), _code(q), _stream()))
+        positions.data_ptr(), _ptr(gate), ld_gate, out.data_ptr(), T, heads, kv_heads, D, DV, int(planes), page_size,
+        float(scale), int(window), int(keep), 1 if plus_one else 0, 1 if gate_channels else 0, _code(q), _stream()))
 
 
-def attention_mma_supports(head_dim: int, page_size: int, group: int) -> bool:
-    return bool(load().xs_attention_mma_supports(head_dim, page_size, group))
+def attention_mma_supports(head_dim: int, page_size: int, group: int, v_dim: int = 0) -> bool:
+    return bool(load().xs_attention_mma_supports(head_dim, v_dim or head_dim, page_size, group))
 
 
-def attention_mma_decode_slots(head_dim: int, tiles: int) -> int:
+def attention_mma_decode_slots(head_dim: int, tiles: int, v_dim: int = 0) -> int:
     """CTAs of the decode attention kernel that run at one time on the device when `tiles` = sequences x kv heads
     (the kernel keeps fewer stages, and so more CTAs an SM, when the tiles alone overfill the device)."""
-    return int(load().xs_attention_mma_decode_slots(head_dim, tiles))
+    return int(load().xs_attention_mma_decode_slots(head_dim, v_dim or head_dim, tiles))
 
 
 def attention_mma_scratch_bytes(rows: int, head_dim: int, splits: int) -> int:
+    """`head_dim`: the values' size."""
     return int(load().xs_attention_mma_scratch_bytes(rows, head_dim, splits))
 
 
@@ -451,37 +487,36 @@ def attention_mma(q: torch.Tensor, pool: torch.Tensor, page_table: torch.Tensor,
                   kv_lens: torch.Tensor, gate: Optional[torch.Tensor], out: torch.Tensor,
                   scratch: Optional[torch.Tensor], n_seqs: int, max_q_len: int, kv_heads: int, page_size: int,
                   scale: float, window: int, splits: int, counters: Optional[torch.Tensor] = None,
-                  bounded_waits: bool = False) -> None:
+                  bounded_waits: bool = False, keep: int = 0, planes: int = 2, plus_one: bool = False,
+                  gate_channels: bool = False) -> None:
     """Tensor-core attention over the paged bfloat16 cache. `scratch`: a byte buffer of at least
     attention_mma_scratch_bytes(tokens * heads, head_dim, splits) when splits > 1. `counters`: at least
     n_seqs * kv_heads zeroed int32 words that the kernel leaves zeroed; with them a decode step (one token a
     sequence) merges its key splits inside the attention kernel instead of in a second one. `bounded_waits`: a decode
     step at head size 64 may take the kernel that the TMA unit feeds; its waits are bounded, and one that gives up sets
-    gemm_tc_status(device), which the caller then has to look at (tc_status_unread)."""
-    _need(q, "q", torch.bfloat16); _need(out, "out", torch.bfloat16); _need(pool, "cache", torch.bfloat16)
+    gemm_tc_status(device), which the caller then has to look at (tc_status_unread). The value size is out's last
+    dimension; `keep` to `gate_channels` as in attention_generic."""
+    _need(q, "q", torch.bfloat16); _need(out, "out", torch.bfloat16)
     _need(page_table, "page table", torch.int32)
     T, heads, D = q.shape
-    if tuple(pool.shape[1:]) != (2, kv_heads, page_size, D):
-        raise KernelError(f"cache is {tuple(pool.shape)}, expected [*, 2, {kv_heads}, {page_size}, {D}]")
-    ld_gate = 0
-    if gate is not None:
-        if gate.dtype != q.dtype or gate.stride(1) != 1 or gate.shape[0] != T or gate.shape[1] < heads:
-            raise KernelError(f"gate is {tuple(gate.shape)} {gate.dtype} for {T} tokens of {heads} heads")
-        ld_gate = gate.stride(0)
+    DV = out.shape[2]
+    _need_pool(pool, kv_heads, page_size, D, DV, planes, torch.bfloat16)
+    ld_gate = _need_gate(gate, q, heads, DV, gate_channels)
     sbytes = 0 if scratch is None else scratch.numel() * scratch.element_size()
     merged = counters is not None and splits > 1 and max_q_len == 1 and heads // kv_heads <= 16
     if merged:
         _need(counters, "counters", torch.int32)
         if counters.numel() < n_seqs * kv_heads:
             raise KernelError(f"attention: {counters.numel()} counters for {n_seqs} sequences of {kv_heads} kv heads")
-    tma = bounded_waits and max_q_len == 1 and D == 64 and heads // kv_heads <= 16
+    tma = bounded_waits and max_q_len == 1 and D == 64 and DV == 64 and heads // kv_heads <= 16
     if tma:
         mark_bounded(q.device)
     _check(load().xs_attention_mma_merged(
         q.data_ptr(), pool.data_ptr(), page_table.data_ptr(), page_table.shape[1], cu_seqlens.data_ptr(),
         kv_lens.data_ptr(), _ptr(gate), ld_gate, out.data_ptr(), _ptr(scratch), sbytes, _ptr(counters) if merged else None,
         pool.shape[0] if tma else 0, gemm_tc_status(q.device).data_ptr() if tma else None,
-        T, n_seqs, max_q_len, heads, kv_heads, D, page_size, float(scale), int(window), int(splits), _stream()),
+        T, n_seqs, max_q_len, heads, kv_heads, D, DV, int(planes), page_size, float(scale), int(window), int(keep),
+        1 if plus_one else 0, 1 if gate_channels else 0, int(splits), _stream()),
         kernels=2 if splits > 1 and not merged else 1)
 
 
@@ -491,25 +526,20 @@ def attention_tc_supports(head_dim: int, page_size: int, group: int) -> bool:
 
 def attention_tc(q: torch.Tensor, pool: torch.Tensor, page_table: torch.Tensor, cu_seqlens: torch.Tensor,
                  kv_lens: torch.Tensor, gate: Optional[torch.Tensor], out: torch.Tensor, n_seqs: int, max_q_len: int,
-                 kv_heads: int, page_size: int, scale: float, window: int, max_kv_len: int = 0) -> None:
+                 kv_heads: int, page_size: int, scale: float, window: int, max_kv_len: int = 0, keep: int = 0,
+                 planes: int = 2, plus_one: bool = False, gate_channels: bool = False) -> None:
     """Attention for prompts on the tcgen05 tensor cores (head size 64): the same operation as attention_mma with
     one key split. A wait that gives up inside the kernel sets gemm_tc_status(device). `max_kv_len` (the longest
     sequence's keys, 0 if unknown) only picks the order in which the kernel's CTAs start."""
-    _need(q, "q", torch.bfloat16); _need(out, "out", torch.bfloat16); _need(pool, "cache", torch.bfloat16)
-    _need(page_table, "page table", torch.int32)
+    _need(q, "q", torch.bfloat16); _need(out, "out", torch.bfloat16); _need(page_table, "page table", torch.int32)
     T, heads, D = q.shape
-    if tuple(pool.shape[1:]) != (2, kv_heads, page_size, D):
-        raise KernelError(f"cache is {tuple(pool.shape)}, expected [*, 2, {kv_heads}, {page_size}, {D}]")
-    ld_gate = 0
-    if gate is not None:
-        if gate.dtype != q.dtype or gate.stride(1) != 1 or gate.shape[0] != T or gate.shape[1] < heads:
-            raise KernelError(f"gate is {tuple(gate.shape)} {gate.dtype} for {T} tokens of {heads} heads")
-        ld_gate = gate.stride(0)
+    _need_pool(pool, kv_heads, page_size, D, out.shape[2], planes, torch.bfloat16)
+    ld_gate = _need_gate(gate, q, heads, D, gate_channels)
     mark_bounded(q.device)
     _check(load().xs_attention_tc(
         q.data_ptr(), pool.data_ptr(), pool.shape[0], page_table.data_ptr(), page_table.shape[1], cu_seqlens.data_ptr(),
-        kv_lens.data_ptr(), _ptr(gate), ld_gate, out.data_ptr(), T, n_seqs, max_q_len, heads, kv_heads, D, page_size,
-        float(scale), int(window), int(max_kv_len), gemm_tc_status(q.device).data_ptr(), _stream()))
+        kv_lens.data_ptr(), _ptr(gate), ld_gate, out.data_ptr(), T, n_seqs, max_q_len, heads, kv_heads, D, int(planes), page_size,
+        float(scale), int(window), int(keep), 1 if plus_one else 0, 1 if gate_channels else 0, int(max_kv_len), gemm_tc_status(q.device).data_ptr(), _stream()))
 
 
 def gemm_small_m_supports(M: int, K: int, ldx: int, ldw: int) -> bool:
@@ -924,11 +954,12 @@ def moe_route(logits: torch.Tensor, top: int, ids: torch.Tensor, wts: torch.Tens
 
 def moe_route_grouped(logits: torch.Tensor, top: int, ids: torch.Tensor, wts: torch.Tensor, experts: Optional[int] = None,
                       correction: Optional[torch.Tensor] = None, groups: int = 1, keep: int = 1, group_top: int = 2,
-                      scale: float = 1.0, renorm: bool = False, score: str = "sigmoid", real: Optional[int] = None) -> None:
+                      scale: float = 1.0, renorm: bool = False, score: str = "sigmoid", real: Optional[int] = None,
+                      renorm_eps: float = 0.0) -> None:
     """Per row of float32 logits: scores s = sigmoid(logit), choice scores c = s + correction; the experts stand in
     `groups` equal groups of neighbours, of which the `keep` with the largest sum of their `group_top` largest choice
     scores stay open; the `top` open experts with the largest c (ties: the lower index) go into ids, their s (times
-    `scale`; divided by their sum with `renorm`) into wts. `score` "softmax": s is the softmax over all `experts` logits
+    `scale`; divided by their sum + `renorm_eps` with `renorm`) into wts. `score` "softmax": s is the softmax over all `experts` logits
     instead. `real`: only the first so many experts have weights; a choice of a later one is written as id -1 (its input
     passes, times its weight)."""
     _need(logits, "router logits", torch.float32); _need(ids, "ids", torch.int32); _need(wts, "weights", torch.float32)
@@ -943,7 +974,7 @@ def moe_route_grouped(logits: torch.Tensor, top: int, ids: torch.Tensor, wts: to
     if ids.numel() < T * top or wts.numel() < T * top:
         raise KernelError(f"moe_route_grouped: {T} tokens x top {top} do not fit ids {ids.numel()} / weights {wts.numel()}")
     _check(load().xs_moe_route_grouped(logits.data_ptr(), ld, T, E, int(top), _ptr(correction), int(groups), int(keep),
-                                       int(group_top), float(scale), 1 if renorm else 0, 1 if score == "softmax" else 0,
+                                       int(group_top), float(scale), 1 if renorm else 0, float(renorm_eps), 1 if score == "softmax" else 0,
                                        E if real is None else int(real), ids.data_ptr(), wts.data_ptr(), _stream()))
 
 
@@ -1383,6 +1414,29 @@ def causal_conv(x: torch.Tensor, taps_w: torch.Tensor, state: torch.Tensor, seq_
                                  cu_seqlens.data_ptr(), slots.data_ptr(), out.data_ptr(), out.stride(0), T, slots.numel(), C,
                                  taps, 1 if act == "silu" else 0, 1 if residual else 0, 1 if all_single else 0, _code(x), _stream()),
            kernels=2 if taps > 1 and not all_single else 1)
+
+
+def poly_norm(z: torch.Tensor, coef: torch.Tensor, out: torch.Tensor, eps: float) -> None:
+    """out = a N(z) + b N(z^2) + c N(z^3) + e per row, (a, b, c, e) = coef and N a division by the row's root mean square."""
+    _need(coef, "coefficients", torch.float32); _need(out, "out", z.dtype)
+    if not z.is_cuda or z.dim() != 2 or z.stride(1) != 1 or coef.numel() != 4 or tuple(out.shape) != tuple(z.shape):
+        raise KernelError(f"poly_norm: z {tuple(z.shape)}, {coef.numel()} coefficients, out {tuple(out.shape)}")
+    T, F_ = z.shape
+    _check(load().xs_poly_norm(z.data_ptr(), z.stride(0), coef.data_ptr(), out.data_ptr(), T, F_, float(eps), _code(z), _stream()))
+
+
+def stream_add(h: torch.Tensor, base: Optional[torch.Tensor] = None, row: Optional[torch.Tensor] = None) -> None:
+    """h [T, n] += base [T, n] + row [n], float32; either may be left out."""
+    _need(h, "h", torch.float32)
+    T, n = h.shape
+    for t, shape, name in ((base, (T, n), "base"), (row, (n,), "row")):
+        if t is not None:
+            _need(t, name, torch.float32)
+            if tuple(t.shape) != shape:
+                raise KernelError(f"stream_add: {name} is {tuple(t.shape)}, expected {shape}")
+    if base is None and row is None:
+        return
+    _check(load().xs_stream_add(h.data_ptr(), _ptr(base), _ptr(row), T, n, _stream()))
 
 
 def gated_add(h: torch.Tensor, branch: torch.Tensor, logits: torch.Tensor, bias: Optional[torch.Tensor] = None) -> None:

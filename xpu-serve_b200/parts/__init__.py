@@ -9,6 +9,7 @@ from .swiglu import SwiGLU
 from .latent_attention import LatentAttentionMixer
 from .mamba2 import Mamba2Mixer
 from .gated_units import ClampedGLU, RoutedExperts, SquaredRelu
+from .poly_norm import PolyNormUnit
 from .mlstm import MLstmMixer
 from .lightning import LightningMixer
 from .gated_delta import GatedDeltaMixer
@@ -20,4 +21,4 @@ __all__ = ["FeedForward", "KVNeed", "Mixer", "Norm", "RMSNorm", "Part", "StateNe
            "AttentionMixer", "ShortConvMixer", "SwiGLU", "Block", "ResidualStream", "LayerNorm", "ScaledRotaryTable",
            "LatentAttentionMixer", "Mamba2Mixer", "ClampedGLU", "RoutedExperts", "SquaredRelu", "MLstmMixer",
            "PairHashEmbedding", "BranchNormBlock", "GatedDeltaMixer", "ParallelMixer", "LearnedPositionEmbedding",
-           "GatedPreNormBlock", "LightningMixer"]
+           "GatedPreNormBlock", "LightningMixer", "PolyNormUnit"]

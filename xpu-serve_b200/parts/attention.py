@@ -10,19 +10,31 @@ gate) only.
 Masks: every earlier key; a sliding window (`window`); or the query's own block of `chunk`
 positions, counted from the sequence's first position (the kernels take one number: 0, W or -C).
 
-Value heads of another size than the key heads (`v_dim`, without rotation): the kernels and
-the cache know one head size, so q, k and v heads are laid out in `padded_head_dim(spec)`
-channels, the surplus rows of their weights (and columns of the output projection) being
-zero: scores and outputs do not change. The per-head norms then see a mean over more
-channels; their eps and weights are scaled so that the result is the norm over head_dim.
+Value heads of another size than the key heads (`v_dim`). v_layout "padded" (without rotation): q, k
+and v heads are laid out in `padded_head_dim(spec)` channels, the surplus rows of their weights (and
+columns of the output projection) being zero: scores and outputs do not change. The per-head norms
+then see a mean over more channels; their eps and weights are scaled so that the result is the norm
+over head_dim. v_layout "own": keys and values each have a size of their own in the kernels and the
+cache, padded in the same way to the next size that the tensor-core kernels take.
+
+Options (config/spec.py: AttentionSpec): a window that keeps the sequence's first positions
+(`keep_first`; the cache keeps their pages); queries and keys of unit root mean square behind the
+rotation (`unit_qk`: a rotation keeps lengths, so the norm is taken in front of it, by the kernel that
+norms, with a weight of ones); keys that are the values (`shared_kv`: one vector a position in the cache,
+loaded once for both products); one added to the softmax's denominator (`plus_one`); a gate on every
+output channel (`out_gate`, in the attention kernels' epilogues); a factor per head on the scores
+(`head_temp`, on the queries as they are stored). A rotation of some of a head's channels, or of
+neighbouring ones, is brought into the kernels' pairing by the order of the weights' rows (`channel_layout`).
 """
 from __future__ import annotations
 
-from typing import Dict
+from dataclasses import replace
+from typing import Dict, List, Tuple
 
 import torch
 
 from .. import registry
+from ..config.spec import RopeSpec, ScaledRopeSpec
 from ..ops import lib as ops
 from .base import KVNeed, Mixer, TensorSpec
 
@@ -44,6 +56,7 @@ def decode_splits(tiles: int, blocks: int, slots: int, fixed: float = 2.0) -> in
 
 
 _TENSOR_CORE_HEAD_DIMS = (16, 32, 48, 64, 96, 128)
+_TENSOR_CORE_VALUE_DIMS = (32, 64, 128)      # beside keys of another size (csrc/attention_pairs.cu)
 
 
 def padded_head_dim(spec) -> int:
@@ -59,13 +72,46 @@ def padded_head_dim(spec) -> int:
     return m + (m & 1)
 
 
-def _pad_heads(t: torch.Tensor, heads: int, d: int, dp: int) -> torch.Tensor:
-    """[heads * d, ...] -> [heads * dp, ...]: every head's rows followed by dp - d zero rows."""
-    if d == dp:
+def head_sizes(spec) -> Tuple[int, int]:
+    """(D, DV): the sizes in which query/key heads and value heads are laid out. "padded": one size for both. "own": the next
+    sizes that the tensor-core kernels take, or (above 128) the next even number."""
+    if spec.v_layout != "own":
+        D = padded_head_dim(spec)
+        return D, D
+    hd, vd = spec.head_dim, spec.v_dim or spec.head_dim
+    D = next((d for d in _TENSOR_CORE_HEAD_DIMS if hd <= d), hd + (hd & 1))
+    if spec.shared_kv:
+        return D, D
+    return D, next((d for d in sorted({D, *_TENSOR_CORE_VALUE_DIMS}) if vd <= d), vd + (vd & 1))
+
+
+def channel_layout(spec, D: int) -> List[int]:
+    """For each of the D channels in which the kernels hold a query or key head: which of the checkpoint's head_dim channels
+    stands there (-1: none, zero). The kernels rotate channels i and i + D/2 together: the two members of each pair that
+    turns go to the same place of the two halves, then the channels that do not turn."""
+    hd, pos = spec.head_dim, spec.position
+    if pos is None:
+        return list(range(hd)) + [-1] * (D - hd)
+    dims = pos.dims if isinstance(pos, ScaledRopeSpec) else hd
+    inter = getattr(pos, "pairing", "half") == "interleaved"
+    first = [2 * i if inter else i for i in range(dims // 2)]
+    second = [2 * i + 1 if inter else i + dims // 2 for i in range(dims // 2)]
+    if not isinstance(pos, ScaledRopeSpec):
+        return first + second                    # (pairs that do not turn have frequency 0 in the table)
+    still = list(range(dims, hd))
+    room = D // 2 - dims // 2
+    a, b = still[:room], still[room:]
+    return first + a + [-1] * (room - len(a)) + second + b + [-1] * (room - len(b))
+
+
+def _arrange_heads(t: torch.Tensor, heads: int, d: int, layout: List[int]) -> torch.Tensor:
+    """[heads * d, ...] -> [heads * len(layout), ...]: every head's rows in the layout's order, zeros where it names none."""
+    if layout == list(range(d)):
         return t
     t = t.reshape(heads, d, *t.shape[1:])
-    pad = torch.zeros(heads, dp - d, *t.shape[2:], dtype=t.dtype)
-    return torch.cat([t, pad], 1).reshape(heads * dp, *t.shape[2:])
+    t = torch.cat([t, torch.zeros(heads, 1, *t.shape[2:], dtype=t.dtype)], 1)
+    at = torch.tensor([c if c >= 0 else d for c in layout])
+    return t[:, at].reshape(heads * len(layout), *t.shape[2:])
 
 
 class AttentionMixer(Mixer):
@@ -78,13 +124,17 @@ class AttentionMixer(Mixer):
         n = spec.names
         vd = spec.v_dim or spec.head_dim
         qd, kd = spec.heads * spec.head_dim, spec.kv_heads * spec.head_dim
+        own_v = spec.own_kv and not spec.shared_kv
         out = {n["q"]: TensorSpec((qd, spec.hidden))}
         if spec.own_kv:
             out[n["k"]] = TensorSpec((kd, spec.hidden))
+        if own_v:
             out[n["v"]] = TensorSpec((spec.kv_heads * vd, spec.hidden))
         out[n["o"]] = TensorSpec((spec.hidden, spec.heads * vd))
         if spec.head_gate:
             out[n["gate"]] = TensorSpec((spec.heads, spec.hidden))
+        if spec.out_gate:
+            out[n["gate"]] = TensorSpec((spec.heads * vd, spec.hidden))
         if spec.qk_norm:
             out[n["q_norm"]] = TensorSpec((spec.head_dim,), init="ones", role="vector")
             if spec.own_kv:
@@ -93,61 +143,84 @@ class AttentionMixer(Mixer):
             out[n["q_bias"]] = TensorSpec((qd,), init="zeros", role="vector")
             if spec.own_kv:
                 out[n["k_bias"]] = TensorSpec((kd,), init="zeros", role="vector")
+            if own_v:
                 out[n["v_bias"]] = TensorSpec((spec.kv_heads * vd,), init="zeros", role="vector")
+        if spec.head_temp:
+            out[n["temp"]] = TensorSpec((spec.heads,), init="uniform:0.5:1.5", role="vector")
         return out
 
     @classmethod
     def cache_need(cls, spec):
         # (a block mask keeps every key: a reader of this cache may have another mask)
-        return KVNeed(spec.kv_heads, padded_head_dim(spec), spec.window if not spec.chunk else 0)
+        D, DV = head_sizes(spec)
+        window = spec.window if not spec.chunk else 0
+        return KVNeed(spec.kv_heads, D, window, planes=1 if spec.shared_kv else 2, keep_first=spec.keep_first if window > 0 else 0,
+                      v_dim=DV if DV != D else 0)
 
     def __init__(self, spec, weights: Dict[str, torch.Tensor], rt):
         vd = spec.v_dim or spec.head_dim
-        D = self.D = padded_head_dim(spec)
-        if D % 2 != 0 or D > 256:
+        D, DV = self.D, self.DV = head_sizes(spec)
+        if D % 2 != 0 or max(D, DV) > 256:
             raise ValueError(f"attention: head sizes {spec.head_dim} / {vd} must be even (or differ) and at most 256")
         if spec.heads % spec.kv_heads != 0:
             raise ValueError(f"attention: {spec.heads} heads over {spec.kv_heads} kv heads")
         if spec.chunk and spec.window:
             raise ValueError("attention: a layer has a window or a block mask, not both")
-        if D != spec.head_dim and spec.position is not None:
+        if spec.shared_kv and vd != spec.head_dim:
+            raise ValueError(f"attention: keys that are the values have one size, not {spec.head_dim} and {vd}")
+        if spec.shared_kv and (spec.position is not None or spec.qk_norm or spec.unit_qk):
+            raise ValueError("attention: keys that are the values as projected are neither rotated nor normed")
+        if D != spec.head_dim and isinstance(spec.position, RopeSpec):
             raise ValueError("attention: value heads of another size than the key heads need a layer without rotation")
+        if spec.qk_norm and spec.unit_qk or spec.head_gate and spec.out_gate:
+            raise ValueError("attention: a layer has learned or unit q/k norms, a gate per head or per channel, not both")
+        if spec.unit_qk and getattr(getattr(spec.position, "scaling", None), "mscale_k", 0.0) != 0.0:
+            raise ValueError("attention: unit queries and keys behind a rotation that changes lengths are not supported")
+        if not spec.scale > 0.0 or spec.keep_first < 0:
+            raise ValueError("attention: the scale must be positive and keep_first not negative")
         self.spec, self.rt = spec, rt
         self.mask = -int(spec.chunk) if spec.chunk else int(spec.window)     # the kernels' one number
         n = spec.names
-        self.q_dim = spec.heads * D
-        self.kv_dim = spec.kv_heads * D
+        self.planes = 1 if spec.shared_kv else 2
+        self.q_dim, self.o_dim = spec.heads * D, spec.heads * DV
+        self.kv_cols = spec.kv_heads * (D + (DV if self.planes == 2 else 0))
+        # what the kernels need beside the window: passed on to each of them
+        self.options = dict(keep=int(spec.keep_first) if spec.window > 0 else 0, planes=self.planes, plus_one=bool(spec.plus_one),
+                            gate_channels=bool(spec.out_gate))
         # the per-head norm over head_dim channels, computed over D: sum / D + eps' = (head_dim / D) (sum / head_dim + eps)
         self.qk_eps = float(spec.qk_norm_eps) * spec.head_dim / D
         norm_scale = (spec.head_dim / D) ** 0.5
-        # A checkpoint whose rotation couples channels 2i and 2i + 1 is brought into the rotate-half order here: within
-        # every head the even channels first, then the odd ones, for q and k alike (their products do not change), and
-        # the per-head norm weights with them.
-        interleaved = spec.position is not None and getattr(spec.position, "pairing", "half") == "interleaved"
-        order = torch.cat([torch.arange(0, D, 2), torch.arange(1, D, 2)]) if interleaved else None
-
-        def per_head(t: torch.Tensor, heads: int) -> torch.Tensor:     # rows (or elements) of q or k, head by head
-            if order is None:
-                return t
-            return t.reshape(heads, D, *t.shape[1:])[:, order].reshape(t.shape)
-
+        # A checkpoint whose rotation couples other channels than i and i + D/2 is brought into that order here, for q and k
+        # alike (their products do not change), and the per-head norm weights with them.
         hd = spec.head_dim
-        wq = _pad_heads(per_head(weights[n["q"]], spec.heads), spec.heads, hd, D)
+        layout = channel_layout(spec, D)
+        v_layout = list(range(vd)) + [-1] * (DV - vd)
+
+        def keys(t: torch.Tensor, heads: int) -> torch.Tensor:         # rows (or elements) of q or k, head by head
+            return _arrange_heads(t, heads, hd, layout)
+
+        def values(t: torch.Tensor, heads: int) -> torch.Tensor:
+            return _arrange_heads(t, heads, vd, v_layout)
+
+        own_v = spec.own_kv and not spec.shared_kv
+        wq = keys(weights[n["q"]], spec.heads)
         q_rows = [wq]
         rows = [wq]
         if spec.own_kv:
-            rows += [_pad_heads(per_head(weights[n["k"]], spec.kv_heads), spec.kv_heads, hd, D),
-                     _pad_heads(weights[n["v"]], spec.kv_heads, vd, D)]
+            rows.append(keys(weights[n["k"]], spec.kv_heads))
+        if own_v:
+            rows.append(values(weights[n["v"]], spec.kv_heads))
         biases = q_biases = None
         if spec.qkv_bias:
-            bq = _pad_heads(per_head(weights[n["q_bias"]], spec.heads), spec.heads, hd, D)
+            bq = keys(weights[n["q_bias"]], spec.heads)
             q_biases = [bq]
             biases = [bq]
             if spec.own_kv:
-                biases += [_pad_heads(per_head(weights[n["k_bias"]], spec.kv_heads), spec.kv_heads, hd, D),
-                           _pad_heads(weights[n["v_bias"]], spec.kv_heads, vd, D)]
-        if spec.head_gate:
-            g = weights[n["gate"]]
+                biases.append(keys(weights[n["k_bias"]], spec.kv_heads))
+            if own_v:
+                biases.append(values(weights[n["v_bias"]], spec.kv_heads))
+        if spec.head_gate or spec.out_gate:
+            g = values(weights[n["gate"]], spec.heads) if spec.out_gate else weights[n["gate"]]
             pad = (-g.shape[0]) % 16      # (whole 16-row tiles: what the few-row product's unpredicated instances and its tails ask for)
             if pad:
                 g = torch.cat([g, torch.zeros(pad, g.shape[1], dtype=g.dtype)], 0)
@@ -162,17 +235,24 @@ class AttentionMixer(Mixer):
             self.b_qkvg = rt.vector(torch.cat([b.to(torch.float32) for b in biases])) if biases is not None else None
         self._q_rows, self._q_biases = q_rows, q_biases          # stacked on the device on the first use as a reader of another cache
         w_o = weights[n["o"]]
-        if D != vd:         # zero columns where the padded value channels stand
-            w_o = _pad_heads(w_o.t().contiguous(), spec.heads, vd, D).t().contiguous()
+        if DV != vd:        # zero columns where the padded value channels stand
+            w_o = values(w_o.t().contiguous(), spec.heads).t().contiguous()
         self.w_o = rt.matrix(w_o)
 
-        def norm_weight(name):
-            return rt.vector(_pad_heads(per_head(weights[name], 1).to(torch.float32), 1, hd, D) * norm_scale)
+        def norm_weight(w: torch.Tensor):
+            return rt.vector(keys(w.to(torch.float32), 1) * norm_scale)
 
-        self.q_norm = norm_weight(n["q_norm"]) if spec.qk_norm else None
-        self.k_norm = norm_weight(n["k_norm"]) if spec.qk_norm and spec.own_kv else None
-        self.position = (registry.position_class(spec.position.kind)(spec.position, rt)
-                         if spec.position is not None else None)
+        self.q_norm = self.k_norm = None
+        if spec.qk_norm:
+            self.q_norm = norm_weight(weights[n["q_norm"]])
+            self.k_norm = norm_weight(weights[n["k_norm"]]) if spec.own_kv else None
+        elif spec.unit_qk:
+            self.q_norm = self.k_norm = norm_weight(torch.ones(hd))
+        self.q_scale = rt.vector(weights[n["temp"]]) if spec.head_temp else None
+        position = spec.position
+        if isinstance(position, ScaledRopeSpec):      # (one table entry per pair of the layout)
+            position = replace(position, head_dim=D)
+        self.position = registry.position_class(position.kind)(position, rt) if position is not None else None
 
     def takes_prenormed(self, rows: int) -> bool:
         return (self.w_qkvg is not None and self.rt.few_rows_shape(rows, self.w_qkvg) and self.w_qkvg.shape[1] % 8 == 0)
@@ -182,11 +262,11 @@ class AttentionMixer(Mixer):
         T = x.shape[0]
         if cache is None or cache.storage is None:
             raise RuntimeError("attention needs a key/value cache")
-        D = self.D
+        D, DV = self.D, self.DV
         if cache.owner:
             if self.w_qkvg is None:
                 raise RuntimeError("attention: a layer without keys and values of its own must read another call's cache")
-            w_in, b_in, gate_at = self.w_qkvg, self.b_qkvg, self.q_dim + 2 * self.kv_dim
+            w_in, b_in, gate_at = self.w_qkvg, self.b_qkvg, self.q_dim + self.kv_cols
         else:
             if self.w_qg is None:
                 self.w_qg = rt.matrix(torch.cat([r.to(torch.float32) for r in self._q_rows], 0))
@@ -196,7 +276,7 @@ class AttentionMixer(Mixer):
         table = step.page_tables[cache.group]
         rope = self.position.table(step.max_positions) if self.position is not None else None
         q = rt.ws.get("attn_q", (T, s.heads, D), rt.act_dtype)
-        if step.decode and rt.rope_behind_product(x, w_in, D):
+        if step.decode and D == DV and self.planes == 2 and self.q_scale is None and rt.rope_behind_product(x, w_in, D):
             # one token a sequence: the per-head norms, the rotation and the cache write run behind the product, in its kernel
             proj = rt.ws.get("attn_qkv", (T, w_in.shape[0]), rt.act_dtype)
             rt.few_rows_rope(x, w_in, proj, b_in, q_out=q, pool=cache.storage if cache.owner else None,
@@ -207,56 +287,59 @@ class AttentionMixer(Mixer):
             proj = rt.linear(x, w_in, "attn_qkv", b_in)
             ops.qk_norm_rope_store(proj, q, cache.storage, table, step.seq_of_token, step.positions, self.q_norm,
                                    self.k_norm, rope, s.heads, s.kv_heads, D, step.page_size, self.qk_eps,
-                                   write_kv=cache.owner)
-        o = rt.ws.get("attn_o", (T, s.heads, D), rt.act_dtype)
-        gate = proj[:, gate_at:] if s.head_gate else None
+                                   write_kv=cache.owner, v_dim=DV, planes=self.planes, q_scale=self.q_scale)
+        o = rt.ws.get("attn_o", (T, s.heads, DV), rt.act_dtype)
+        gate = proj[:, gate_at:] if s.head_gate or s.out_gate else None
         self.attend(q, cache, table, step, gate, o)
         if into is not None:
-            return into.product(o.view(T, self.q_dim), self.w_o)
-        return rt.linear(o.view(T, self.q_dim), self.w_o, "mixer_out")
+            return into.product(o.view(T, self.o_dim), self.w_o)
+        return rt.linear(o.view(T, self.o_dim), self.w_o, "mixer_out")
 
     def attend(self, q, cache, table, step, gate, o) -> None:
-        s, rt, D, mask = self.spec, self.rt, self.D, self.mask
-        if step.fixed_shape and rt.mode == "bfloat16" and ops.attention_mma_supports(D, step.page_size, s.heads // s.kv_heads):
+        s, rt, D, DV, mask = self.spec, self.rt, self.D, self.DV, self.mask
+        group = s.heads // s.kv_heads
+        mma = rt.mode == "bfloat16" and ops.attention_mma_supports(D, step.page_size, group, DV)
+        tc = mma and rt.prompt_attention == "tcgen05" and D == DV and ops.attention_tc_supports(D, step.page_size, group)
+        if step.fixed_shape and mma:
             # a step captured for any lengths up to its bounds: one key split, grids from the bounds
-            if rt.prompt_attention == "tcgen05" and ops.attention_tc_supports(D, step.page_size, s.heads // s.kv_heads):
+            if tc:
                 ops.attention_tc(q, cache.storage, table, step.cu_seqlens, step.kv_lens, gate, o, step.n_seqs,
-                                 step.max_q_len, s.kv_heads, step.page_size, s.scale, mask, step.max_kv_len)
+                                 step.max_q_len, s.kv_heads, step.page_size, s.scale, mask, step.max_kv_len, **self.options)
             else:
                 ops.attention_mma(q, cache.storage, table, step.cu_seqlens, step.kv_lens, gate, o, None, step.n_seqs,
-                                  step.max_q_len, s.kv_heads, step.page_size, s.scale, mask, 1)
+                                  step.max_q_len, s.kv_heads, step.page_size, s.scale, mask, 1, **self.options)
             return
-        if rt.mode == "bfloat16" and ops.attention_mma_supports(D, step.page_size, s.heads // s.kv_heads):
+        if mma:
             # Few tiles and long key ranges (decoding): split each range over several CTAs so that
             # every SM streams a part of the cache; the partial results meet in scratch memory.
-            tokens_per_tile = 64 // (s.heads // s.kv_heads)
+            tokens_per_tile = 64 // group
             tiles = sum(-(-int(n) // tokens_per_tile) for n in step.q_lens_host) * s.kv_heads
             blocks = -(-step.max_kv_len // step.page_size)
             if s.window > 0 or s.chunk > 0:       # the keys a tile can see span at most so many pages
-                blocks = min(blocks, -(-(max(s.window, s.chunk) + step.max_q_len) // step.page_size) + 1)
-            if step.decode and s.heads // s.kv_heads <= 16 and rt.attn_split_factor == 0:
-                splits = decode_splits(tiles, blocks, max(1, ops.attention_mma_decode_slots(D, tiles)),
+                blocks = min(blocks, -(-(max(s.window, s.chunk) + step.max_q_len) // step.page_size) + 1
+                             + -(-self.options["keep"] // step.page_size))
+            if step.decode and group <= 16 and rt.attn_split_factor == 0:
+                splits = decode_splits(tiles, blocks, max(1, ops.attention_mma_decode_slots(D, tiles, DV)),
                                        rt.attn_fixed_cost)
             else:
                 splits = max(1, min(blocks, 32, (max(rt.attn_split_factor, 1) * rt.sm_count) // max(tiles, 1)))
             # prompts: the tcgen05 kernel, unless few tiles face many keys (a short piece of a long sequence), where
             # cutting the keys over more CTAs is worth more
-            if ((splits == 1 or step.max_kv_len <= 512) and not step.decode and rt.prompt_attention == "tcgen05"
-                    and ops.attention_tc_supports(D, step.page_size, s.heads // s.kv_heads)):
+            if tc and (splits == 1 or step.max_kv_len <= 512) and not step.decode:
                 ops.attention_tc(q, cache.storage, table, step.cu_seqlens, step.kv_lens, gate, o, step.n_seqs,
-                                 step.max_q_len, s.kv_heads, step.page_size, s.scale, mask, step.max_kv_len)
+                                 step.max_q_len, s.kv_heads, step.page_size, s.scale, mask, step.max_kv_len, **self.options)
                 return
             scratch = None
             if splits > 1:
-                need = ops.attention_mma_scratch_bytes(q.shape[0] * s.heads, D, splits)
+                need = ops.attention_mma_scratch_bytes(q.shape[0] * s.heads, DV, splits)
                 scratch = rt.ws.get("attn_scratch", (need,), torch.uint8)
             counters = rt.attn_counters if (rt.fuse_tails and rt.tail_attn and step.n_seqs * s.kv_heads <= rt.attn_counters.numel()) else None
             ops.attention_mma(q, cache.storage, table, step.cu_seqlens, step.kv_lens, gate, o, scratch, step.n_seqs,
                               step.max_q_len, s.kv_heads, step.page_size, s.scale, mask, splits, counters=counters,
-                              bounded_waits=step.decode)
+                              bounded_waits=step.decode, **self.options)
             return
         ops.attention_generic(q, cache.storage, table, step.seq_of_token, step.positions, gate, o, s.kv_heads,
-                              step.page_size, s.scale, mask)
+                              step.page_size, s.scale, mask, **self.options)
 
 
 registry.register_mixer(AttentionMixer.kind, AttentionMixer)

@@ -51,12 +51,15 @@ class TensorSpec:
 
 @dataclass(frozen=True)
 class KVNeed:
-    """Keys and values for every cached position (window 0) or the last `window` of them. `planes` 1: one vector
-    a position and head instead of a key and a value (a latent from which both are made)."""
+    """Keys and values for every cached position (window 0) or the last `window` of them and the first `keep_first`.
+    `planes` 1: one vector a position and head instead of a key and a value (a latent from which both are made, or keys
+    that are the values too). `v_dim`: size of a value when it differs from the key's (0: head_dim)."""
     kv_heads: int
     head_dim: int
     window: int = 0
     planes: int = 2
+    keep_first: int = 0
+    v_dim: int = 0
 
 
 @dataclass(frozen=True)

@@ -23,6 +23,7 @@ weights, rt), forward(stream, step, cache, next_norm), first_norm.
 """
 from __future__ import annotations
 
+from dataclasses import replace
 from typing import Dict, Optional, Tuple
 
 import torch
@@ -125,6 +126,10 @@ class ResidualStream:
             self._pending = None
             self._pre = None
 
+    def changed(self) -> None:
+        """`h` is about to be rewritten in place (after `flush`): nothing prepared from its old values may be used."""
+        self._pre = None
+
     def replace(self, h: torch.Tensor) -> None:
         """The stream becomes `h` (float32, same shape): what a step does that rewrites the stream between layers."""
         self.flush()
@@ -208,7 +213,7 @@ class TokenSide:
         self.w_gate = rt.matrix(weights[n["gate"]])
         self.w_proj = rt.matrix(weights[n["proj"]])
         # (an RMS norm with a plain weight, whatever the model's own norm is)
-        self.norm = registry.norm_class("rmsnorm")(NormSpec(width, spec.eps), weights, n["norm"], rt)
+        self.norm = registry.norm_class("rmsnorm")(NormSpec(width, spec.eps, scale=spec.scale), weights, n["norm"], rt)
 
     def forward(self, stream: "ResidualStream", step) -> None:
         rt = self.rt
@@ -255,12 +260,14 @@ class Block:
         norm_cls = registry.norm_class(spec.norm.kind)
         self.pre_mixer = norm_cls(spec.norm, weights, n["pre_mixer"], rt)
         self.pre_ffn = norm_cls(spec.norm, weights, n["pre_ffn"], rt) if self.ffn is not None else None
-        self.post_mixer = norm_cls(spec.norm, weights, n["post_mixer"], rt) if spec.sandwich else None
-        self.post_ffn = norm_cls(spec.norm, weights, n["post_ffn"], rt) if spec.sandwich and self.ffn is not None else None
+        # (a constant on the branches, branch_scale, is part of the norms behind them)
+        post = spec.norm if spec.branch_scale == 1.0 else replace(spec.norm, scale=spec.norm.scale * spec.branch_scale)
+        if spec.branch_scale != 1.0 and not (spec.sandwich and spec.norm.kind == "rmsnorm"):
+            raise ValueError("pre_norm: a constant on the branches needs RMS norms behind them (sandwich)")
+        self.post_mixer = norm_cls(post, weights, n["post_mixer"], rt) if spec.sandwich else None
+        self.post_ffn = norm_cls(post, weights, n["post_ffn"], rt) if spec.sandwich and self.ffn is not None else None
         self.first_norm = self.pre_mixer      # the norm that reads the stream first: what the block before may prepare
         self.side = TokenSide(spec.token_side, weights, rt, spec.norm.width) if getattr(spec, "token_side", None) is not None else None
-        if self.side is not None and spec.sandwich:
-            raise ValueError("pre_norm: a token-side input behind sandwich norms is not supported")
 
     def forward(self, stream: ResidualStream, step, cache, next_norm: Optional[Norm] = None) -> None:
         """`next_norm`: the norm that reads the stream after this block (the next block's first, or the

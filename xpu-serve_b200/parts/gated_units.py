@@ -13,7 +13,7 @@ RoutedExperts:  `experts` gated feed-forwards without biases (SwiGLU, or clamped
                 groups of neighbouring experts, weighted by the scores as they are (config/spec.py: RoutedExpertsSpec).
                 `activation` "relu_squared": an expert is down(max(up x, 0)^2).
                 `score` "softmax_all": scores softmax over all router outputs, chosen by score plus a correction, weighted
-                by the scores as they are; with `identity` the router's last outputs stand for the token's input itself
+                by the scores as they are or over their sum; with `identity` the router's last outputs stand for the token's input itself
                 (such a choice takes no place in the plan; the combine kernel adds weight times input).
 """
 from __future__ import annotations
@@ -114,7 +114,8 @@ class RoutedExperts(FeedForward):
             out[n["correction"]] = TensorSpec((outputs,), init="uniform:-0.3:0.3", role="vector")
         if spec.shared is not None:
             out.update(registry.ffn_class(spec.shared.kind).tensors(spec.shared))
-            out[n["shared_gate"]] = TensorSpec((1, spec.hidden))
+            if spec.shared_gated:
+                out[n["shared_gate"]] = TensorSpec((1, spec.hidden))
         return out
 
     def __init__(self, spec, weights: Dict[str, torch.Tensor], rt):
@@ -126,10 +127,11 @@ class RoutedExperts(FeedForward):
         if self.identity < 0 or (self.identity > 0 and spec.score != "softmax_all"):
             raise ValueError("routed experts: identity outputs belong to softmax_all scores")
         if spec.score == "softmax" and (spec.correction or spec.groups != 1):
-            raise ValueError("routed experts: a correction and groups belong to sigmoid scores")
-        if spec.groups < 1 or spec.experts % spec.groups != 0 or not 1 <= spec.keep_groups <= spec.groups \
-                or spec.keep_groups * (spec.experts // spec.groups) + self.identity < spec.top:
-            raise ValueError(f"routed experts: {spec.experts} experts in {spec.groups} groups of which {spec.keep_groups} stay open "
+            raise ValueError("routed experts: a correction and groups belong to sigmoid scores or to the softmax over all outputs")
+        outputs = spec.experts + self.identity
+        if spec.groups < 1 or outputs % spec.groups != 0 or not 1 <= spec.keep_groups <= spec.groups \
+                or spec.keep_groups * (outputs // spec.groups) < spec.top:
+            raise ValueError(f"routed experts: {outputs} outputs in {spec.groups} groups of which {spec.keep_groups} stay open "
                              f"cannot give {spec.top} choices")
         self.spec, self.rt = spec, rt
         self.gated = spec.activation == "gated"
@@ -155,7 +157,8 @@ class RoutedExperts(FeedForward):
         self.shared = None
         if spec.shared is not None:
             # the shared unit's gate logit is one more row of the router product (its float32 sums serve both)
-            router = torch.cat([router, weights[n["shared_gate"]].to(torch.float32).reshape(1, H)], 0)
+            if spec.shared_gated:
+                router = torch.cat([router, weights[n["shared_gate"]].to(torch.float32).reshape(1, H)], 0)
             self.shared = registry.ffn_class(spec.shared.kind)(spec.shared, weights, rt)
         self.w_router = rt.matrix(router)
         self.correction = rt.vector(weights[n["correction"]]) if spec.correction else None
@@ -169,7 +172,7 @@ class RoutedExperts(FeedForward):
         logits = ws.get("moe_logits", (T, self.w_router.shape[0]), torch.float32)
         ops.moe_logits(y, self.w_router, logits)            # float32 sums of the activation type's products, not rounded
         outputs = s.experts + self.identity
-        shared_gate = logits[:, outputs:] if shared is not None else None
+        shared_gate = logits[:, outputs:] if shared is not None and s.shared_gated else None
         ids = ws.get("moe_ids", (n,), torch.int32)
         wts = ws.get("moe_wts", (n,), torch.float32)
         place = ws.get("moe_place", (n,), torch.int32)
@@ -177,10 +180,12 @@ class RoutedExperts(FeedForward):
         meta = ws.get("moe_meta", (4 + 3 * ops.moe_max_tiles(n, s.experts),), torch.int32)
         if s.score == "softmax_all":
             ops.moe_route_grouped(logits, s.top, ids, wts, experts=outputs, correction=self.correction, scale=s.route_scale,
-                                  score="softmax", real=s.experts)
+                                  score="softmax", real=s.experts, groups=s.groups, keep=s.keep_groups,
+                                  group_top=s.group_top, renorm=s.renorm, renorm_eps=s.renorm_eps)
         elif s.score == "sigmoid":
             ops.moe_route_grouped(logits, s.top, ids, wts, experts=s.experts, correction=self.correction, groups=s.groups,
-                                  keep=s.keep_groups, group_top=s.group_top, scale=s.route_scale, renorm=s.renorm)
+                                  keep=s.keep_groups, group_top=s.group_top, scale=s.route_scale, renorm=s.renorm,
+                                  renorm_eps=s.renorm_eps)
         else:
             ops.moe_route(logits, s.top, ids, wts, experts=s.experts, scale=s.route_scale)
         out = ws.get("ffn_out", (T, s.hidden), rt.act_dtype)

@@ -22,7 +22,10 @@ class RMSNorm(Norm):
         super().__init__(spec, weights, weight_name, rt)
         # (a weight stored around zero: the norm multiplies by offset + w, formed once in float32)
         offset = float(getattr(spec, "offset", 0.0))
-        self.w = rt.vector(weights[weight_name].to(torch.float32) + offset if offset else weights[weight_name])
+        w = weights[weight_name].to(torch.float32) + offset if offset else weights[weight_name]
+        # (a constant on the norm's result is part of the weight)
+        scale = float(getattr(spec, "scale", 1.0))
+        self.w = rt.vector(w.to(torch.float32) * scale if scale != 1.0 else w)
         self.eps = float(spec.eps)
 
     def normed(self, x: torch.Tensor) -> torch.Tensor:

@@ -16,6 +16,7 @@ from __future__ import annotations
 import torch
 
 from .. import registry
+from ..config.spec import BandRopeScalingSpec
 
 
 class RotaryTable:
@@ -49,22 +50,27 @@ class RotaryTable:
 
 
 class ScaledRotaryTable:
-    """The table of a rotation over the first `dims` channels of a vector (pair i couples channels i and i + dims/2),
-    with frequencies stretched for long sequences (config/spec.py: ScaledRopeSpec, RopeScalingSpec):
+    """The table of a rotation over the first `dims` channels of a vector, with frequencies stretched for long sequences
+    (config/spec.py: ScaledRopeSpec). RopeScalingSpec:
 
         f_i = theta^(-2i/dims);  where(t) = dims * ln(original / (2 pi t)) / (2 ln theta)
         lo = max(floor(where(fast)), 0);  hi = min(ceil(where(slow)), dims - 1)
         ramp_i = clamp((i - lo) / max(hi - lo, 0.001), 0, 1);  f'_i = f_i / factor * ramp_i + f_i * (1 - ramp_i)
 
-    and cos and sin multiplied by mscale_k * ln(factor) + 1. Angles are formed in float64 as RotaryTable's are.
-    table(n) is [n or more, dims / 2, 2] float32."""
+    and cos and sin multiplied by mscale_k * ln(factor) + 1. BandRopeScalingSpec, with l_i = 2 pi / f_i:
+
+        s_i = clamp((original / l_i - low) / (high - low), 0, 1);  f'_i = (1 - s_i) f_i / factor + s_i f_i
+
+    Angles are formed in float64 as RotaryTable's are. table(n) is [n or more, head_dim / 2, 2] float32, (1, 0) for the
+    pairs behind the first dims / 2."""
     kind = "rope_scaled"
 
     def __init__(self, spec, rt):
         self.spec, self.rt = spec, rt
         sc = spec.scaling
-        self.key = ("rope_scaled", spec.dims, float(spec.theta),
-                    None if sc is None else (sc.factor, sc.original, sc.fast, sc.slow, sc.mscale_k))
+        if spec.dims % 2 != 0 or not 0 < spec.dims <= spec.head_dim:
+            raise ValueError(f"rotation over {spec.dims} of {spec.head_dim} channels (an even number is needed)")
+        self.key = ("rope_scaled", spec.head_dim, spec.dims, float(spec.theta), sc)
 
     def frequencies(self):
         """(float64 [dims / 2], the factor on cos and sin)."""
@@ -75,6 +81,10 @@ class ScaledRotaryTable:
         sc = s.scaling
         if sc is None:
             return f, 1.0
+        if isinstance(sc, BandRopeScalingSpec):
+            ratio = sc.original * f / (2.0 * math.pi)          # original / wavelength
+            s = torch.clamp((ratio - sc.low) / (sc.high - sc.low), 0.0, 1.0)
+            return (1.0 - s) * f / sc.factor + s * f, 1.0
 
         def where(turns: float) -> float:
             return s.dims * math.log(sc.original / (2.0 * math.pi * turns)) / (2.0 * math.log(s.theta))
@@ -92,6 +102,11 @@ class ScaledRotaryTable:
         pos = torch.arange(n_positions, dtype=torch.float64, device=self.rt.device)
         angle = pos[:, None] * f.to(self.rt.device)[None, :]
         table = (torch.stack([torch.cos(angle), torch.sin(angle)], dim=-1) * m).to(torch.float32).contiguous()
+        still = self.spec.head_dim // 2 - self.spec.dims // 2
+        if still > 0:
+            rest = torch.zeros((n_positions, still, 2), dtype=torch.float32, device=self.rt.device)
+            rest[..., 0] = 1.0
+            table = torch.cat([table, rest], 1).contiguous()
         if have is not None:     # a captured graph may still read the shorter table: keep it alive
             self.rt.shared.setdefault(("kept",), []).append(have)
         self.rt.shared[self.key] = table

@@ -29,6 +29,8 @@ def expected_tensors(spec: ModelSpec, prefix: Optional[str] = None) -> Dict[str,
         out[spec.names["head"]] = TensorSpec((spec.vocab, spec.hidden))
     if spec.mixes_in:
         out[p + spec.names["pass_in"]] = TensorSpec((spec.hidden, 2 * spec.hidden))
+    if spec.pass_steps:
+        out[p + spec.names["pass_step"]] = TensorSpec((spec.pass_steps, spec.hidden), role="vector")
     for name, shape in spec.shared_tables().items():
         out[p + name] = TensorSpec(tuple(shape))
     for layer in spec.layers:
