@@ -125,14 +125,16 @@ class ScaledRopeSpec:
     """A rotation of the first `dims` channels of a vector of `head_dim` channels: pair i couples channels i and
     i + dims/2 (not i + head_dim/2), or with `pairing` "interleaved" channels 2i and 2i + 1, and turns by
     pos * theta^(-2i/dims), scaled as `scaling` says (a RopeScalingSpec or a BandRopeScalingSpec; None: as is). The table
-    has head_dim/2 entries a position, the identity behind the first dims/2. The kernels know one pairing, i and
-    i + head_dim/2 of the vector they are given: a mixer whose checkpoint pairs otherwise reorders its weights' rows."""
+    has `pairs` entries a position (0: dims/2), the identity behind the first dims/2. The attention kernels know one
+    pairing, i and i + D/2 of a vector of D channels with D/2 entries: a mixer whose checkpoint pairs otherwise reorders its
+    weights' rows."""
     head_dim: int
     theta: float
     dims: int
     scaling: Optional[object] = None
     kind: str = "rope_scaled"
     pairing: str = "half"
+    pairs: int = 0
 
 
 @dataclass(frozen=True)

@@ -251,7 +251,7 @@ class AttentionMixer(Mixer):
         self.q_scale = rt.vector(weights[n["temp"]]) if spec.head_temp else None
         position = spec.position
         if isinstance(position, ScaledRopeSpec):      # (one table entry per pair of the layout)
-            position = replace(position, head_dim=D)
+            position = replace(position, pairs=D // 2)
         self.position = registry.position_class(position.kind)(position, rt) if position is not None else None
 
     def takes_prenormed(self, rows: int) -> bool:

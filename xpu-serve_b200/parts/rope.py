@@ -61,8 +61,8 @@ class ScaledRotaryTable:
 
         s_i = clamp((original / l_i - low) / (high - low), 0, 1);  f'_i = (1 - s_i) f_i / factor + s_i f_i
 
-    Angles are formed in float64 as RotaryTable's are. table(n) is [n or more, head_dim / 2, 2] float32, (1, 0) for the
-    pairs behind the first dims / 2."""
+    Angles are formed in float64 as RotaryTable's are. table(n) is [n or more, `pairs` or dims / 2, 2] float32, (1, 0)
+    for the pairs behind the first dims / 2."""
     kind = "rope_scaled"
 
     def __init__(self, spec, rt):
@@ -70,7 +70,7 @@ class ScaledRotaryTable:
         sc = spec.scaling
         if spec.dims % 2 != 0 or not 0 < spec.dims <= spec.head_dim:
             raise ValueError(f"rotation over {spec.dims} of {spec.head_dim} channels (an even number is needed)")
-        self.key = ("rope_scaled", spec.head_dim, spec.dims, float(spec.theta), sc)
+        self.key = ("rope_scaled", max(spec.pairs, spec.dims // 2), spec.dims, float(spec.theta), sc)
 
     def frequencies(self):
         """(float64 [dims / 2], the factor on cos and sin)."""
@@ -102,7 +102,7 @@ class ScaledRotaryTable:
         pos = torch.arange(n_positions, dtype=torch.float64, device=self.rt.device)
         angle = pos[:, None] * f.to(self.rt.device)[None, :]
         table = (torch.stack([torch.cos(angle), torch.sin(angle)], dim=-1) * m).to(torch.float32).contiguous()
-        still = self.spec.head_dim // 2 - self.spec.dims // 2
+        still = self.spec.pairs - self.spec.dims // 2
         if still > 0:
             rest = torch.zeros((n_positions, still, 2), dtype=torch.float32, device=self.rt.device)
             rest[..., 0] = 1.0
