@@ -229,6 +229,53 @@ def run_vekuzen_stacks(batch: int, steps: int, warmup: int, only=None) -> int:
     return run_stacks("vekuzen", VEKUZEN_STACKS, vekuzen_stack_configs, batch, steps, warmup, only)
 
 
+# Gararax layer stacks (`--workload gararax`; random weights), each beside the closest existing stack of equal width, layer
+# count and vocabulary: unit-norm attention under a window that keeps the first 64 positions, behind a PolyNorm unit of 8,192
+# (which holds what a SwiGLU of 5,504 holds), beside LFM3's sliding-window attention; keys that are the values under the same
+# window, beside Nimelorn's attention of the same head sizes under a block mask; keys of 128 with values of 32 over every
+# earlier position, beside Nimelorn's attention with 128 for both and a block as long as the context; the last two with routed
+# experts and a shared unit. Every Gararax layer also reads its slice of the second token table, and the first stack starts
+# with the vector that a pass over repeated layers starts with.
+def _windowed(heads, kv_heads, dim, vdim, size, keep, rot=None):
+    m = {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "scale": dim ** -0.5, "mask": {"size": size, "keep_first": keep}}
+    if rot:
+        m["rot"] = rot
+    return m
+
+
+_G_MOE = {"kind": "moe", "expert": {"ff": 1024}, "router": {"experts": 16, "identity": 2, "top": 4, "groups": {"count": 3, "keep": 2}},
+          "shared": {"ff": 1024}}
+GARARAX_STACKS = {
+    "normed_dense": (([("attention", _windowed(32, 8, 64, 64, 1024, 64, {"base": 10000.0, "dims": 64, "scaling": {
+        "factor": 8.0, "low": 1.0, "high": 4.0, "original": 8192}}), {"kind": "dense", "ff": 8192})] * 2, {"start": 0, "stop": 2, "times": 1}),
+                     ("nimelorn beside", "blocked_dense")),
+    "shared_values_experts": (([("attention_2", _windowed(32, 8, 64, 64, 1024, 64), _G_MOE)] * 2, None),
+                              ("nimelorn", [("attention", _blocked(32, 8, 64, 64, 1024), _N_MOE)] * 2)),
+    "tempered_experts": (([("attention_3", {"heads": 16, "kv_heads": 4, "dim": 128, "vdim": 32, "scale": 128 ** -0.5,
+                                            "rot": {"base": 500000.0, "dims": 64}}, _G_MOE)] * 2, None),
+                         ("nimelorn", [("attention", _blocked(16, 4, 128, 128, CONTEXT), _N_MOE)] * 2)),
+}
+
+
+def gararax_stack_configs(name: str, width: int = 2048, vocab: int = 32768):
+    from xpu_serve_b200.config import GararaxConfig, NimelornConfig
+    (layers, loop), beside = GARARAX_STACKS[name]
+    ours = {"architecture": "Gararax", "width": width, "vocab": vocab, "norm": {"eps": 1e-5}, "residual_mult": 0.5,
+            "token_side": {"dim": 256}, "layers": [{"type": t, "mixer": m, "mlp": f} for t, m, f in layers]}
+    if loop:
+        ours["loop"] = loop
+    if beside[0] == "nimelorn beside":          # (the LFM3 stack that stands beside a Nimelorn stack)
+        return GararaxConfig.from_json(ours), nimelorn_stack_configs(beside[1], width, vocab)[1]
+    other = {"architecture": "Nimelorn", "width": width, "vocab": vocab, "norm": {"eps": 1e-5},
+             "embedding": {"scale": float(width) ** 0.5, "bigram": {"buckets": 65521, "mul_prev": 8191, "mul_cur": 31}},
+             "layers": [{"type": t, "mixer": m, "mlp": f} for t, m, f in beside[1]]}
+    return GararaxConfig.from_json(ours), ("nimelorn", NimelornConfig.from_json(other))
+
+
+def run_gararax_stacks(batch: int, steps: int, warmup: int, only=None) -> int:
+    return run_stacks("gararax", GARARAX_STACKS, gararax_stack_configs, batch, steps, warmup, only)
+
+
 def run_stacks(workload: str, stacks, configs_of, batch: int, steps: int, warmup: int, only=None) -> int:
     """Prefill (one prompt of 2,048 tokens in one step) and decode (batch 8 after 2,048-token prompts, CUDA graph) of
     each stack of the workload and of the stack beside it, device-timed as the headline's points are. With XS_PROFILE=1
@@ -595,8 +642,8 @@ def main() -> int:
                          "at long context), which the default run adds to `points`")
     ap.add_argument("--only", default=None, choices=["decode", "prefill", "sample"],
                     help="time one part only and print a short line (for profiler captures)")
-    ap.add_argument("--stacks", default=None, help="with --workload saralix, nimelorn, tozarax or vekuzen: a comma list of the stacks to run (all)")
-    ap.add_argument("--workload", default=None, choices=sorted(WORKLOADS) + ["saralix", "nimelorn", "tozarax", "vekuzen"],
+    ap.add_argument("--stacks", default=None, help="with --workload saralix, nimelorn, tozarax, vekuzen or gararax: a comma list of the stacks to run (all)")
+    ap.add_argument("--workload", default=None, choices=sorted(WORKLOADS) + ["saralix", "nimelorn", "tozarax", "vekuzen", "gararax"],
                     help="instead of the default run: a batch of unequal prompts at another shape of the family")
     args = ap.parse_args()
 
@@ -614,6 +661,8 @@ def main() -> int:
         return run_saralix_stacks(args.batch or 8, args.steps or 128, args.warmup, args.stacks.split(",") if args.stacks else None)
     if args.workload == "nimelorn":
         return run_nimelorn_stacks(args.batch or 8, args.steps or 128, args.warmup, args.stacks.split(",") if args.stacks else None)
+    if args.workload == "gararax":
+        return run_gararax_stacks(args.batch or 8, args.steps or 128, args.warmup, args.stacks.split(",") if args.stacks else None)
     if args.workload == "vekuzen":
         return run_vekuzen_stacks(args.batch or 8, args.steps or 128, args.warmup, args.stacks.split(",") if args.stacks else None)
     if args.workload == "tozarax":

@@ -140,11 +140,11 @@ class AttentionMixer(Mixer):
             if spec.own_kv:
                 out[n["k_norm"]] = TensorSpec((spec.head_dim,), init="ones", role="vector")
         if spec.qkv_bias:
-            out[n["q_bias"]] = TensorSpec((qd,), init="zeros", role="vector")
+            out[n["q_bias"]] = TensorSpec((qd,), role="vector")
             if spec.own_kv:
-                out[n["k_bias"]] = TensorSpec((kd,), init="zeros", role="vector")
+                out[n["k_bias"]] = TensorSpec((kd,), role="vector")
             if own_v:
-                out[n["v_bias"]] = TensorSpec((spec.kv_heads * vd,), init="zeros", role="vector")
+                out[n["v_bias"]] = TensorSpec((spec.kv_heads * vd,), role="vector")
         if spec.head_temp:
             out[n["temp"]] = TensorSpec((spec.heads,), init="uniform:0.5:1.5", role="vector")
         return out
