@@ -97,9 +97,9 @@ __global__ void qk_norm_rope_store_kernel(const T* __restrict__ qkv, int64_t ld,
     }
 }
 
-// bfloat16, head sizes 16, 32, 64, 128, 256: a thread owns 8 neighbouring channels (one 16-byte load and
-// store), the D / 8 threads of a head are neighbours in a warp; the sum of squares and the partner channels
-// (i and i + D / 2 sit D / 16 lanes apart) travel by shuffles.
+// bfloat16, head sizes 16, 32, 48, 64, 96, 128, 256: a thread owns 8 neighbouring channels (one 16-byte load and
+// store), the D / 8 threads of a head are neighbours in a warp (a warp holds as many whole heads as fit); the sum of
+// squares and the partner channels (i and i + D / 2 sit D / 16 lanes apart) travel by shuffles.
 template <int D>
 __global__ void __launch_bounds__(256) qk_norm_rope_store_vec_kernel(
     const __nv_bfloat16* __restrict__ qkv, int64_t ld, __nv_bfloat16* __restrict__ q_out, __nv_bfloat16* __restrict__ pool,
@@ -108,6 +108,8 @@ __global__ void __launch_bounds__(256) qk_norm_rope_store_vec_kernel(
     const float2* __restrict__ rope, int Tn, int Hq, int Hkv, int DV, int planes, const float* __restrict__ q_scale,
     int page_size, float eps, int write_kv) {
     constexpr int G = D / 8;        // threads of a head
+    constexpr int heads_a_warp = 32 / G;
+    constexpr bool pow2 = (G & (G - 1)) == 0;
     constexpr int half = D / 2;
     pdl_launch_dependents();
     // Positions, page numbers, norm weights and the rotation table are not written by the kernel before this one
@@ -115,10 +117,10 @@ __global__ void __launch_bounds__(256) qk_norm_rope_store_vec_kernel(
     // (value channels are walked D at a time whatever the value heads' size: a thread's 8 lie inside one head)
     const int v_cols = write_kv && planes > 1 ? Hkv * DV : 0;
     const int heads_total = Hq + (write_kv ? Hkv : 0) + (v_cols + D - 1) / D;
-    const int64_t thread = (int64_t)blockIdx.x * blockDim.x + threadIdx.x;
-    const int64_t item = thread / G;
-    const int part = (int)(thread % G);
-    bool live = item < (int64_t)Tn * heads_total;           // dead threads still take part in the shuffles
+    const int lane = threadIdx.x & 31, part = lane % G;
+    const int64_t item = ((int64_t)blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5)) * heads_a_warp + lane / G;
+    // (dead threads, and a warp's lanes behind its last whole head, still take part in the shuffles)
+    bool live = lane / G < heads_a_warp && item < (int64_t)Tn * heads_total;
     const int t = live ? (int)(item / heads_total) : 0;
     const int hh = live ? (int)(item % heads_total) : 0;
     const int pos = positions[t];
@@ -178,8 +180,15 @@ __global__ void __launch_bounds__(256) qk_norm_rope_store_vec_kernel(
     float ss = 0.0f;
 #pragma unroll
     for (int j = 0; j < 8; ++j) ss += x[j] * x[j];
+    if constexpr (pow2) {
 #pragma unroll
-    for (int o = G / 2; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+        for (int o = G / 2; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+    } else {                     // every thread of a head adds the head's terms in the same order
+        float sum = 0.0f;
+#pragma unroll
+        for (int o = 0; o < G; ++o) sum += __shfl_sync(0xffffffffu, ss, (lane - part + o) & 31);
+        ss = sum;
+    }
     if (rotate && w != nullptr) {
         const float inv = 1.0f / sqrtf(ss / (float)D + eps);
 #pragma unroll
@@ -188,7 +197,10 @@ __global__ void __launch_bounds__(256) qk_norm_rope_store_vec_kernel(
     // the partner's 8 channels: i + D/2 for the lower half, i - D/2 for the upper half
     float y[8];
 #pragma unroll
-    for (int j = 0; j < 8; ++j) y[j] = G > 1 ? __shfl_xor_sync(0xffffffffu, x[j], G / 2) : 0.0f;
+    for (int j = 0; j < 8; ++j) {
+        if constexpr (pow2) y[j] = G > 1 ? __shfl_xor_sync(0xffffffffu, x[j], G / 2) : 0.0f;
+        else y[j] = __shfl_sync(0xffffffffu, x[j], (lane - part + (part + G / 2) % G) & 31);
+    }
     if (rotate && rope != nullptr) {
 #pragma unroll
         for (int j = 0; j < 8; ++j) {
@@ -310,13 +322,13 @@ XS_API int xs_qk_norm_rope_store(const void* qkv, int64_t ld, void* q_out, void*
     XS_REQUIRE(Hq > 0 && Hkv > 0 && Hq % Hkv == 0, "qk_norm_rope: %d heads over %d kv heads", Hq, Hkv);
     XS_REQUIRE(!write_kv || (pool != nullptr && page_table != nullptr && P > 0), "qk_norm_rope: no cache to write to");
     const int64_t items = (int64_t)T * (Hq + (write_kv ? planes * Hkv : 0));
-    // bfloat16 with 16-byte rows everywhere and a head size whose halves sit a power of two of lanes apart
-    const bool vec = dtype == XS_BF16 && (D == 16 || D == 32 || D == 64 || D == 128 || D == 256) && DV % 8 == 0 && ld % 8 == 0 &&
+    // bfloat16 with 16-byte rows everywhere and a head size that has an instance
+    const bool vec = dtype == XS_BF16 && (D == 16 || D == 32 || D == 48 || D == 64 || D == 96 || D == 128 || D == 256) && DV % 8 == 0 && ld % 8 == 0 &&
                      (uintptr_t)qkv % 16 == 0 && (uintptr_t)q_out % 16 == 0 && (!write_kv || (uintptr_t)pool % 16 == 0) &&
                      (q_w == nullptr || (uintptr_t)q_w % 16 == 0) && (k_w == nullptr || (uintptr_t)k_w % 16 == 0);
     if (vec) {
         const int64_t vitems = (int64_t)T * (Hq + (write_kv ? Hkv : 0) + (write_kv && planes > 1 ? ceil_div_i((int64_t)Hkv * DV, D) : 0));
-        const int vblocks = ceil_div_i(vitems * (D / 8), 256);
+        const int vblocks = ceil_div_i(ceil_div_i(vitems, 32 / (D / 8)), 8);       // 8 warps a block
 #define XS_ROPE_VEC(DD)                                                                                            \
     xs_launch(qk_norm_rope_store_vec_kernel<DD>, dim3(vblocks), dim3(256), 0, stream, (const __nv_bfloat16*)qkv, ld, \
               (__nv_bfloat16*)q_out, (__nv_bfloat16*)pool, page_table, P, seq_of_token, positions, q_w, k_w,        \
@@ -324,7 +336,9 @@ XS_API int xs_qk_norm_rope_store(const void* qkv, int64_t ld, void* q_out, void*
         switch (D) {
             case 16: XS_ROPE_VEC(16); break;
             case 32: XS_ROPE_VEC(32); break;
+            case 48: XS_ROPE_VEC(48); break;
             case 64: XS_ROPE_VEC(64); break;
+            case 96: XS_ROPE_VEC(96); break;
             case 128: XS_ROPE_VEC(128); break;
             default: XS_ROPE_VEC(256); break;
         }

@@ -543,6 +543,7 @@ XS_API int xs_attention_mma_merged(const void* q, const void* pool, const int32_
     const int G = Hq / Hkv;
     XS_REQUIRE(xs_attention_mma_supports(D, DV, page_size, G),
                "attention (tensor cores): head sizes %d / %d, page size %d, group %d is not supported", D, DV, page_size, G);
+    XS_REQUIRE(gate == nullptr || !gate_channels || (ld_gate % 2 == 0 && (uintptr_t)gate % 4 == 0), "attention: a gate per channel needs 4-byte rows");
     XS_REQUIRE((planes == 2 || (planes == 1 && D == DV)) && keep >= 0 && scale > 0.0f, "attention: %d planes, %d kept, scale %g", planes, keep, (double)scale);
     XS_REQUIRE(splits >= 1 && splits <= 64 && max_q_len >= 1 && n_seqs >= 1 && P >= 1,
                "attention: bad sizes (1 to 64 key splits)");

@@ -303,12 +303,19 @@ __global__ void __launch_bounds__(NTHREADS, prompt_ctas(D, DV)) attention_mma_ke
             float f = inv_denominator(l, m, p.plus_one);
             if (p.gate != nullptr && !p.gate_channels) f *= gate_of(p, t, h);
             __nv_bfloat16* dst = p.out + row * DV + (lane & 3) * 2;
+            __nv_bfloat162 gates[DTILES];        // (all asked for before the first is used)
+            if (p.gate_channels) {
+                const __nv_bfloat16* from = p.gate + (int64_t)t * p.ld_gate + h * DV + (lane & 3) * 2;
+#pragma unroll
+                for (int i = 0; i < DTILES; ++i) gates[i] = *reinterpret_cast<const __nv_bfloat162*>(from + i * 8);
+            }
 #pragma unroll
             for (int i = 0; i < DTILES; ++i) {
                 float g0 = f, g1 = f;
                 if (p.gate_channels) {
-                    g0 *= gate_of(p, t, h * DV + i * 8 + (lane & 3) * 2);
-                    g1 *= gate_of(p, t, h * DV + i * 8 + (lane & 3) * 2 + 1);
+                    const float2 z = __bfloat1622float2(gates[i]);
+                    g0 = __fdividef(f, 1.0f + __expf(-z.x));
+                    g1 = __fdividef(f, 1.0f + __expf(-z.y));
                 }
                 *reinterpret_cast<__nv_bfloat162*>(dst + i * 8) =
                     __floats2bfloat162_rn(o[i][half * 2] * g0, o[i][half * 2 + 1] * g1);
