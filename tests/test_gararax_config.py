@@ -103,6 +103,10 @@ def test_how_heads_are_laid_out():
     assert [head_sizes(l.mixer) for l in A.layers] == [(16, 32), (16, 16), (16, 16), (16, 16)]
     assert [head_sizes(l.mixer) for l in B.layers] == [(128, 32), (64, 64), (64, 64), (96, 64)]
     assert [head_sizes(l.mixer) for l in W.layers] == [(160, 128), (48, 136)]
+    big = copy.deepcopy(tiny.CONFIGS["B"])                     # both above 32 and at most 64: 64
+    big["layers"][1]["mixer"].update(dim=40, vdim=56)
+    big["layers"][2]["mixer"].update(dim=36, vdim=36)
+    assert [head_sizes(l.mixer) for l in GararaxConfig.from_json(big).model_spec().layers[1:3]] == [(64, 64)] * 2
     # neighbours 2i and 2i + 1 (all twelve channels turn) and halves of the first eight channels go to places i and i + 8
     assert channel_layout(A.layers[0].mixer, 16) == [0, 2, 4, 6, 8, 10, -1, -1, 1, 3, 5, 7, 9, 11, -1, -1]
     assert channel_layout(A.layers[2].mixer, 16) == [0, 1, 2, 3, 8, 9, 10, 11, 4, 5, 6, 7, 12, 13, -1, -1]

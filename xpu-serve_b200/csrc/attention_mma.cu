@@ -70,7 +70,7 @@ __global__ void __launch_bounds__(160) attention_decode_tma_kernel(const __grid_
     unsigned char* k_sm = base;                                              // [NST][64][128 bytes], swizzled
     const bool own_v = p.planes > 1;                                         // (else the keys' rows serve as the values')
     unsigned char* v_sm = own_v ? base + NST * kPageBytes : base;
-    __nv_bfloat16* q_sm = reinterpret_cast<__nv_bfloat16*>(base + 2 * NST * kPageBytes);      // [16][LD]
+    __nv_bfloat16* q_sm = reinterpret_cast<__nv_bfloat16*>(base + (own_v ? 2 : 1) * NST * kPageBytes);      // [16][LD]
     __shared__ __align__(8) uint64_t bar_full[NST], bar_empty[NST];
     __shared__ float sm_m[4][QROWS], sm_l[4][QROWS];
     __shared__ int pages_sm[64];
@@ -419,12 +419,17 @@ int g_attn_tma_stages = 3;
 // 1.16 ms against 1.27) want the fourth CTA more. 0: always the driver's choice.
 int g_attn_tma_carveout = 72;
 
+// Shared memory of the TMA-fed kernel: stages of keys and (planes 2) values, the queries.
+size_t tma_smem(int stages, int planes) {
+    return (size_t)(planes == 1 ? 1 : 2) * stages * BN * 64 * sizeof(__nv_bfloat16) + (size_t)16 * 72 * sizeof(__nv_bfloat16) + 1024;
+}
+
 template <int NST, bool KEEP_L1>
 int launch_decode_tma_as(const AttnParams& p, const CUtensorMap& map, int* status, int n_seqs, cudaStream_t stream) {
-    const size_t smem = (size_t)2 * NST * BN * 64 * sizeof(__nv_bfloat16) + (size_t)16 * 72 * sizeof(__nv_bfloat16) + 1024;
+    const size_t smem = tma_smem(NST, p.planes);
     static bool opted = false;
     if (!opted) {
-        cudaFuncSetAttribute(attention_decode_tma_kernel<NST, KEEP_L1>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        cudaFuncSetAttribute(attention_decode_tma_kernel<NST, KEEP_L1>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)tma_smem(NST, 2));
         if (KEEP_L1)
             cudaFuncSetAttribute(attention_decode_tma_kernel<NST, KEEP_L1>, cudaFuncAttributePreferredSharedMemoryCarveout,
                                  g_attn_tma_carveout);
@@ -468,17 +473,17 @@ XS_API int xs_attention_mma_set_decode_stages(int n) {
 // CTAs of the decode kernel (one token a sequence) that run at one time on this device when `tiles` = sequences x kv
 // heads (the number of stages, and with it the CTAs an SM, follows from that); 0 when the head size is not
 // supported. The caller sizes its key splits by it.
-XS_API int xs_attention_mma_decode_slots(int D, int DV, int64_t tiles) {
+XS_API int xs_attention_mma_decode_slots(int D, int DV, int planes, int64_t tiles) {
     if (D != DV) return pair_decode_slots(D, DV, tiles);
     if (D == 64 && g_attn_decode_tma && encode_fn() != nullptr) {       // the TMA-fed kernel: its own occupancy
-        static int per_sm[8][2] = {};
-        const int n = g_attn_tma_stages, k = tma_keeps_l1(tiles) ? 1 : 0;
-        if (per_sm[n][k] == 0) {
-            const size_t smem = (size_t)2 * n * BN * 64 * sizeof(__nv_bfloat16) + (size_t)16 * 72 * sizeof(__nv_bfloat16) + 1024;
+        static int per_sm[8][2][2] = {};
+        const int n = g_attn_tma_stages, k = tma_keeps_l1(tiles) ? 1 : 0, own = planes > 1 ? 1 : 0;
+        if (per_sm[n][k][own] == 0) {
+            const size_t smem = tma_smem(n, planes);
             int got = 0;
 #define XS_TMA_OCC(NST, KEEP)                                                                                                \
     do {                                                                                                                     \
-        cudaFuncSetAttribute(attention_decode_tma_kernel<NST, KEEP>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
+        cudaFuncSetAttribute(attention_decode_tma_kernel<NST, KEEP>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)tma_smem(NST, 2)); \
         if (KEEP)                                                                                                            \
             cudaFuncSetAttribute(attention_decode_tma_kernel<NST, KEEP>, cudaFuncAttributePreferredSharedMemoryCarveout,     \
                                  g_attn_tma_carveout);                                                                       \
@@ -496,9 +501,9 @@ XS_API int xs_attention_mma_decode_slots(int D, int DV, int64_t tiles) {
 #undef XS_TMA_OCC
             // (the occupancy query may not know of the carveout: 164 KB hold three CTAs of three stages)
             if (k && got > (int)((size_t)g_attn_tma_carveout * 228 * 1024 / 100 / (smem + 1024))) got = (int)((size_t)g_attn_tma_carveout * 228 * 1024 / 100 / (smem + 1024));
-            per_sm[n][k] = got > 0 ? got : 1;
+            per_sm[n][k][own] = got > 0 ? got : 1;
         }
-        return sm_count() * per_sm[n][k];
+        return sm_count() * per_sm[n][k][own];
     }
     switch (D) {
         case 16: return decode_slots<16, 16>(tiles);

@@ -108,7 +108,7 @@ def _signatures(lib) -> None:
     lib.xs_attention_tc_supports.restype = c_int
     lib.xs_attention_tc_supports.argtypes = [c_int, c_int, c_int]
     lib.xs_attention_mma_decode_slots.restype = c_int
-    lib.xs_attention_mma_decode_slots.argtypes = [c_int, c_int, c_int64]
+    lib.xs_attention_mma_decode_slots.argtypes = [c_int, c_int, c_int, c_int64]
     lib.xs_gemm_small_m_supports.restype = c_int
     lib.xs_gemm_small_m_supports.argtypes = [c_int, c_int, c_int64, c_int64]
     lib.xs_gemm_tc_supports.restype = c_int
@@ -472,10 +472,10 @@ def attention_mma_supports(head_dim: int, page_size: int, group: int, v_dim: int
     return bool(load().xs_attention_mma_supports(head_dim, v_dim or head_dim, page_size, group))
 
 
-def attention_mma_decode_slots(head_dim: int, tiles: int, v_dim: int = 0) -> int:
+def attention_mma_decode_slots(head_dim: int, tiles: int, v_dim: int = 0, planes: int = 2) -> int:
     """CTAs of the decode attention kernel that run at one time on the device when `tiles` = sequences x kv heads
     (the kernel keeps fewer stages, and so more CTAs an SM, when the tiles alone overfill the device)."""
-    return int(load().xs_attention_mma_decode_slots(head_dim, v_dim or head_dim, tiles))
+    return int(load().xs_attention_mma_decode_slots(head_dim, v_dim or head_dim, planes, tiles))
 
 
 def attention_mma_scratch_bytes(rows: int, head_dim: int, splits: int) -> int:

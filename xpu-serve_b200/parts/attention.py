@@ -74,11 +74,15 @@ def padded_head_dim(spec) -> int:
 
 def head_sizes(spec) -> Tuple[int, int]:
     """(D, DV): the sizes in which query/key heads and value heads are laid out. "padded": one size for both. "own": the next
-    sizes that the tensor-core kernels take, or (above 128) the next even number."""
+    sizes that the tensor-core kernels take, or (above 128) the next even number. Both above 32 and at most 64 become 64, the
+    size that the tcgen05 kernel of prompts and the TMA-fed kernel of single tokens take (48 and 64, 16 heads over 4, 2,048
+    tokens: the mma.sync kernel at 48 / 64 takes longer than the tcgen05 kernel at 64 / 64)."""
     if spec.v_layout != "own":
         D = padded_head_dim(spec)
         return D, D
     hd, vd = spec.head_dim, spec.v_dim or spec.head_dim
+    if 32 < hd <= 64 and 32 < vd <= 64:
+        return 64, 64
     D = next((d for d in _TENSOR_CORE_HEAD_DIMS if hd <= d), hd + (hd & 1))
     if spec.shared_kv:
         return D, D
@@ -319,7 +323,7 @@ class AttentionMixer(Mixer):
                 blocks = min(blocks, -(-(max(s.window, s.chunk) + step.max_q_len) // step.page_size) + 1
                              + -(-self.options["keep"] // step.page_size))
             if step.decode and group <= 16 and rt.attn_split_factor == 0:
-                splits = decode_splits(tiles, blocks, max(1, ops.attention_mma_decode_slots(D, tiles, DV)),
+                splits = decode_splits(tiles, blocks, max(1, ops.attention_mma_decode_slots(D, tiles, DV, self.planes)),
                                        rt.attn_fixed_cost)
             else:
                 splits = max(1, min(blocks, 32, (max(rt.attn_split_factor, 1) * rt.sm_count) // max(tiles, 1)))
