@@ -403,8 +403,9 @@ def test_attention_kernels(kernel, shape, window, keep, plus_one, gated):
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
 @pytest.mark.parametrize("H,G,D,DV,planes", [(4, 2, 16, 32, 2), (8, 1, 128, 32, 2), (3, 3, 48, 64, 2), (2, 2, 64, 64, 1), (5, 1, 64, 128, 2), (2, 1, 6, 10, 2),
                                              (2, 2, 32, 48, 2), (1, 1, 256, 8, 2)])
-def test_norm_rotation_and_store(H, G, D, DV, planes, dtype):
-    """Queries normed, rotated and multiplied by their head's factor; keys normed, rotated and written with the raw values into
+@pytest.mark.parametrize("biased", [False, True])
+def test_norm_rotation_and_store(biased, H, G, D, DV, planes, dtype):
+    """Columns with a bias (or none): queries normed, rotated and multiplied by their head's factor; keys normed, rotated and written with the raw values into
     pages whose values have another size (or none): nothing else of the cache changes."""
     from xpu_serve_b200.ops import lib as ops
     rng = np.random.default_rng(D + DV)
@@ -418,10 +419,12 @@ def test_norm_rotation_and_store(H, G, D, DV, planes, dtype):
     w = torch.from_numpy(rng.uniform(0.5, 1.5, D)).float()
     rope = torch.from_numpy(rng.standard_normal((200, D // 2, 2))).float()
     temp = torch.from_numpy(rng.uniform(-1.5, 1.5, H)).float()
+    bias = torch.from_numpy(rng.standard_normal(cols + 8)).float() if biased else None
     q = torch.empty(T, H, D, dtype=dtype, device="cuda")
     ops.qk_norm_rope_store(x.cuda()[:, :cols], q, pool, table.cuda(), dev_i32(seq_of), dev_i32(positions), w.cuda(), w.cuda(), rope.cuda(),
-                           H, G, D, page, eps, True, v_dim=DV, planes=planes, q_scale=temp.cuda())
-    xd, r, half = x.double().numpy(), rope.double().numpy(), D // 2
+                           H, G, D, page, eps, True, v_dim=DV, planes=planes, q_scale=temp.cuda(),
+                           bias=bias.cuda() if biased else None)
+    xd, r, half = x.double().numpy() + (bias.double().numpy() if biased else 0.0), rope.double().numpy(), D // 2
 
     def turn(rows):                 # [T, n, D]
         y = plain.unit_rms(rows, eps) * w.double().numpy()
@@ -438,10 +441,11 @@ def test_norm_rotation_and_store(H, G, D, DV, planes, dtype):
         p = int(table[seq_of[t], positions[t] // page])
         k_view[p, :, positions[t] % page] = torch.from_numpy(want_k[t]).to(dtype)
         if planes == 2:
-            v_view.view(6, G, page, DV)[p, :, positions[t] % page] = x[t, (H + G) * D:cols].view(G, DV)
+            v_view.view(6, G, page, DV)[p, :, positions[t] % page] = torch.from_numpy(xd[t, (H + G) * D:cols]).to(dtype).view(G, DV)
     got, want = pool.double().cpu().numpy().reshape(6, -1), flat.double().numpy()
     assert np.abs(got - want).max() <= tol * np.abs(want).max()
-    assert np.array_equal(got[:, G * page * D:], want[:, G * page * D:])          # values as they are
+    if not biased:
+        assert np.array_equal(got[:, G * page * D:], want[:, G * page * D:])      # values as they are
     touched = np.zeros((6, G, page, D), dtype=bool)
     for t in range(T):
         touched[int(table[seq_of[t], positions[t] // page]), :, positions[t] % page] = True
@@ -470,7 +474,7 @@ def test_poly_norm_alone(F, dtype):
     assert (gap <= tol).all(), gap
 
 
-@pytest.mark.parametrize("E,identity,top,groups,keep", [(5, 1, 2, 2, 1), (16, 2, 4, 2, 1), (7, 2, 3, 3, 2), (8, 0, 1, 1, 1), (40, 24, 6, 8, 3), (60, 4, 8, 4, 4), (200, 56, 16, 16, 2)])
+@pytest.mark.parametrize("E,identity,top,groups,keep", [(5, 1, 2, 2, 1), (16, 2, 4, 2, 1), (7, 2, 3, 3, 2), (8, 0, 1, 1, 1), (40, 24, 6, 8, 3), (60, 4, 8, 4, 4), (200, 56, 16, 16, 2), (60, 4, 29, 2, 1)])
 def test_routing_kernel_alone(E, identity, top, groups, keep):
     """Choices and weights against the oracle's wherever the choice is no close call; corrections of both signs, so that open
     groups hold negative choice scores."""

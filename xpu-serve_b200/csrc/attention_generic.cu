@@ -22,7 +22,7 @@ __global__ void qk_norm_rope_store_kernel(const T* __restrict__ qkv, int64_t ld,
                                           const int32_t* __restrict__ positions, const float* __restrict__ q_w,
                                           const float* __restrict__ k_w, const float2* __restrict__ rope, int Tn,
                                           int Hq, int Hkv, int D, int DV, int planes, const float* __restrict__ q_scale,
-                                          int page_size, float eps, int write_kv) {
+                                          const float* __restrict__ bias, int page_size, float eps, int write_kv) {
     pdl_launch_dependents();
     pdl_wait();
     const int heads_total = Hq + (write_kv ? planes * Hkv : 0);
@@ -34,7 +34,8 @@ __global__ void qk_norm_rope_store_kernel(const T* __restrict__ qkv, int64_t ld,
     const int half = D >> 1;
     const int pos = positions[t];
     // q heads and k heads (D each), then v heads (DV each) are consecutive
-    const T* src = qkv + (int64_t)t * ld + (int64_t)hh * D;
+    int64_t col = (int64_t)hh * D;
+    const T* src = qkv + (int64_t)t * ld + col;
 
     T* dst;
     const float* w;
@@ -50,9 +51,10 @@ __global__ void qk_norm_rope_store_kernel(const T* __restrict__ qkv, int64_t ld,
         const int page = page_table[(int64_t)seq * P + pos / page_size];
         T* at = pool + (int64_t)page * Hkv * page_size * (planes == 1 ? D : D + DV);
         if (which == 1) {   // values: a plain copy
-            src = qkv + (int64_t)t * ld + (int64_t)(Hq + Hkv) * D + (int64_t)kvh * DV;
+            col = (int64_t)(Hq + Hkv) * D + (int64_t)kvh * DV;
+            src = qkv + (int64_t)t * ld + col;
             dst = at + (int64_t)Hkv * page_size * D + ((int64_t)kvh * page_size + pos % page_size) * DV;
-            for (int d = lane; d < DV; d += 32) dst[d] = src[d];
+            for (int d = lane; d < DV; d += 32) dst[d] = bias == nullptr ? src[d] : from_f32<T>(to_f32(src[d]) + bias[col + d]);
             return;
         }
         dst = at + ((int64_t)kvh * page_size + pos % page_size) * D;
@@ -67,6 +69,10 @@ __global__ void qk_norm_rope_store_kernel(const T* __restrict__ qkv, int64_t ld,
         if (i < half) {
             a[u] = to_f32(src[i]);
             b[u] = to_f32(src[i + half]);
+            if (bias != nullptr) {
+                a[u] += bias[col + i];
+                b[u] += bias[col + i + half];
+            }
             ss += a[u] * a[u] + b[u] * b[u];
         }
     }
@@ -106,7 +112,7 @@ __global__ void __launch_bounds__(256) qk_norm_rope_store_vec_kernel(
     const int32_t* __restrict__ page_table, int P, const int32_t* __restrict__ seq_of_token,
     const int32_t* __restrict__ positions, const float* __restrict__ q_w, const float* __restrict__ k_w,
     const float2* __restrict__ rope, int Tn, int Hq, int Hkv, int DV, int planes, const float* __restrict__ q_scale,
-    int page_size, float eps, int write_kv) {
+    const float* __restrict__ bias, int page_size, float eps, int write_kv) {
     constexpr int G = D / 8;        // threads of a head
     constexpr int heads_a_warp = 32 / G;
     constexpr bool pow2 = (G & (G - 1)) == 0;
@@ -158,6 +164,14 @@ __global__ void __launch_bounds__(256) qk_norm_rope_store_vec_kernel(
         wv[4] = w1.x; wv[5] = w1.y; wv[6] = w1.z; wv[7] = w1.w;
     }
     const bool low = c0 < half;
+    float bv[8];
+#pragma unroll
+    for (int j = 0; j < 8; ++j) bv[j] = 0.0f;
+    if (bias != nullptr && live) {
+        const float4 b0 = *reinterpret_cast<const float4*>(bias + hh * D + c0), b1 = *reinterpret_cast<const float4*>(bias + hh * D + c0 + 4);
+        bv[0] = b0.x; bv[1] = b0.y; bv[2] = b0.z; bv[3] = b0.w;
+        bv[4] = b1.x; bv[5] = b1.y; bv[6] = b1.z; bv[7] = b1.w;
+    }
     float2 cs[8];
     if (rotate && rope != nullptr) {
         const float2* at = rope + (int64_t)pos * half + (low ? c0 : c0 - half);
@@ -173,8 +187,8 @@ __global__ void __launch_bounds__(256) qk_norm_rope_store_vec_kernel(
 #pragma unroll
         for (int j = 0; j < 4; ++j) {
             const float2 f = __bfloat1622float2(h2[j]);
-            x[2 * j] = f.x;
-            x[2 * j + 1] = f.y;
+            x[2 * j] = f.x + bv[2 * j];
+            x[2 * j + 1] = f.y + bv[2 * j + 1];
         }
     }
     float ss = 0.0f;
@@ -210,7 +224,7 @@ __global__ void __launch_bounds__(256) qk_norm_rope_store_vec_kernel(
         }
     }
     if (!live) return;
-    if (rotate) {
+    if (rotate || bias != nullptr) {
         uint4 o;
         __nv_bfloat162* h2 = reinterpret_cast<__nv_bfloat162*>(&o);
 #pragma unroll
@@ -310,11 +324,12 @@ __global__ void attention_generic_kernel(const T* __restrict__ q, const T* __res
 }  // namespace
 
 // planes 2: keys of D and values of DV channels a head; 1: keys only (they are the values too; DV is then D).
-// q_scale (or null): a float32 factor per query head, applied last.
+// q_scale (or null): a float32 factor per query head, applied last. bias (or null): a float32 number per column of qkv, added
+// first, to the values too (16-byte aligned).
 XS_API int xs_qk_norm_rope_store(const void* qkv, int64_t ld, void* q_out, void* pool, const int32_t* page_table,
                                  int P, const int32_t* seq_of_token, const int32_t* positions, const float* q_w,
                                  const float* k_w, const float* rope, int T, int Hq, int Hkv, int D, int DV, int planes,
-                                 const float* q_scale, int page_size, float eps, int write_kv, int dtype,
+                                 const float* q_scale, const float* bias, int page_size, float eps, int write_kv, int dtype,
                                  cudaStream_t stream) {
     if (T == 0) return 0;
     XS_REQUIRE(D > 0 && D % 2 == 0 && D <= kMaxHeadDim, "qk_norm_rope: head size %d (even, at most %d)", D, kMaxHeadDim);
@@ -325,14 +340,14 @@ XS_API int xs_qk_norm_rope_store(const void* qkv, int64_t ld, void* q_out, void*
     // bfloat16 with 16-byte rows everywhere and a head size that has an instance
     const bool vec = dtype == XS_BF16 && (D == 16 || D == 32 || D == 48 || D == 64 || D == 96 || D == 128 || D == 256) && DV % 8 == 0 && ld % 8 == 0 &&
                      (uintptr_t)qkv % 16 == 0 && (uintptr_t)q_out % 16 == 0 && (!write_kv || (uintptr_t)pool % 16 == 0) &&
-                     (q_w == nullptr || (uintptr_t)q_w % 16 == 0) && (k_w == nullptr || (uintptr_t)k_w % 16 == 0);
+                     (q_w == nullptr || (uintptr_t)q_w % 16 == 0) && (k_w == nullptr || (uintptr_t)k_w % 16 == 0) && (uintptr_t)bias % 16 == 0;
     if (vec) {
         const int64_t vitems = (int64_t)T * (Hq + (write_kv ? Hkv : 0) + (write_kv && planes > 1 ? ceil_div_i((int64_t)Hkv * DV, D) : 0));
         const int vblocks = ceil_div_i(ceil_div_i(vitems, 32 / (D / 8)), 8);       // 8 warps a block
 #define XS_ROPE_VEC(DD)                                                                                            \
     xs_launch(qk_norm_rope_store_vec_kernel<DD>, dim3(vblocks), dim3(256), 0, stream, (const __nv_bfloat16*)qkv, ld, \
               (__nv_bfloat16*)q_out, (__nv_bfloat16*)pool, page_table, P, seq_of_token, positions, q_w, k_w,        \
-              (const float2*)rope, T, Hq, Hkv, DV, planes, q_scale, page_size, eps, write_kv)
+              (const float2*)rope, T, Hq, Hkv, DV, planes, q_scale, bias, page_size, eps, write_kv)
         switch (D) {
             case 16: XS_ROPE_VEC(16); break;
             case 32: XS_ROPE_VEC(32); break;
@@ -350,7 +365,7 @@ XS_API int xs_qk_norm_rope_store(const void* qkv, int64_t ld, void* q_out, void*
     XS_DISPATCH_DTYPE(dtype, TT,
                       xs_launch(qk_norm_rope_store_kernel<TT>, dim3(blocks), dim3(128), 0, stream,
                           (const TT*)qkv, ld, (TT*)q_out, (TT*)pool, page_table, P, seq_of_token, positions, q_w,
-                          k_w, (const float2*)rope, T, Hq, Hkv, D, DV, planes, q_scale, page_size, eps, write_kv));
+                          k_w, (const float2*)rope, T, Hq, Hkv, D, DV, planes, q_scale, bias, page_size, eps, write_kv));
     XS_LAUNCH_CHECK("qk_norm_rope_store");
     return 0;
 }

@@ -592,8 +592,8 @@ XS_API int xs_moe_route_grouped(const float* logits, int ld, int T, int E, int t
                                 int group_top, float scale, int renorm, float renorm_eps, int score, int real, int32_t* ids,
                                 float* wts, cudaStream_t stream) {
     if (T == 0) return 0;
-    XS_REQUIRE(T > 0 && E > 0 && top > 0 && top <= E && top <= kMaxTop && ld >= E,
-               "moe_route_grouped: %d tokens, %d experts (row stride %d), top %d (at most %d)", T, E, ld, top, kMaxTop);
+    XS_REQUIRE(T > 0 && E > 0 && top > 0 && top <= E && top <= 32 && ld >= E,
+               "moe_route_grouped: %d tokens, %d experts (row stride %d), top %d (at most 32: a lane a choice)", T, E, ld, top);
     XS_REQUIRE(groups > 0 && E % groups == 0 && keep > 0 && keep <= groups && group_top > 0 && group_top <= 8,
                "moe_route_grouped: %d experts in %d groups of which %d are kept (a group's %d largest count)", E, groups, keep, group_top);
     XS_REQUIRE((int64_t)keep * (E / groups) >= top, "moe_route_grouped: %d groups of %d experts cannot give %d choices", keep, E / groups, top);

@@ -44,7 +44,7 @@ def _signatures(lib) -> None:
         "xs_lightning_scan": [P, L, I, I, I, P, P, P, P, P, I, I, I, I, I, P, P, I, P, P],
         "xs_zero_rows": [P, P, I, L, P],
         "xs_gemm_generic": [P, P, P, P, I, I, I, I, I, L, L, L, P],
-        "xs_qk_norm_rope_store": [P, L, P, P, P, I, P, P, P, P, P, I, I, I, I, I, I, P, I, F, I, I, P],
+        "xs_qk_norm_rope_store": [P, L, P, P, P, I, P, P, P, P, P, I, I, I, I, I, I, P, P, I, F, I, I, P],
         "xs_attention_generic": [P, P, P, I, P, P, P, L, P, I, I, I, I, I, I, I, F, I, I, I, I, I, P],
         "xs_short_conv": [P, L, P, P, P, P, P, P, P, I, I, I, I, I, I, P],
         "xs_attention_mma": [P, P, P, I, P, P, P, L, P, P, L, I, I, I, I, I, I, I, F, I, I, P],
@@ -414,10 +414,11 @@ def qk_norm_rope_store(qkv: torch.Tensor, q_out: torch.Tensor, pool: Optional[to
                        page_table: Optional[torch.Tensor], seq_of_token: torch.Tensor, positions: torch.Tensor,
                        q_w: Optional[torch.Tensor], k_w: Optional[torch.Tensor], rope: Optional[torch.Tensor],
                        heads: int, kv_heads: int, head_dim: int, page_size: int, eps: float, write_kv: bool,
-                       v_dim: int = 0, planes: int = 2, q_scale: Optional[torch.Tensor] = None) -> None:
+                       v_dim: int = 0, planes: int = 2, q_scale: Optional[torch.Tensor] = None,
+                       bias: Optional[torch.Tensor] = None) -> None:
     """Columns [q heads | k heads | v heads] of qkv: per-head norms and rotation of q (to q_out, times `q_scale` [heads] when
     given) and k, and keys and values into the cache's pages. `v_dim` (0: head_dim) is a value head's size; planes 1: there
-    are no values."""
+    are no values. `bias`: a number per column, added first, to the values too (where the product could not add it)."""
     v_dim = v_dim or head_dim
     _need(q_out, "q_out", qkv.dtype)
     if qkv.stride(1) != 1:
@@ -438,6 +439,10 @@ def qk_norm_rope_store(qkv: torch.Tensor, q_out: torch.Tensor, pool: Optional[to
         _need(q_scale, "q_scale", torch.float32)
         if q_scale.numel() != heads:
             raise KernelError(f"q_scale has {q_scale.numel()} elements for {heads} heads")
+    if bias is not None:
+        _need(bias, "bias", torch.float32)
+        if bias.numel() < width:
+            raise KernelError(f"a bias of {bias.numel()} for {width} columns")
     if rope is not None:
         _need(rope, "rope table", torch.float32)
         if tuple(rope.shape[1:]) != (head_dim // 2, 2):
@@ -445,7 +450,7 @@ def qk_norm_rope_store(qkv: torch.Tensor, q_out: torch.Tensor, pool: Optional[to
     P = 0 if page_table is None else page_table.shape[1]
     _check(load().xs_qk_norm_rope_store(
         qkv.data_ptr(), qkv.stride(0), q_out.data_ptr(), _ptr(pool), _ptr(page_table), P, seq_of_token.data_ptr(),
-        positions.data_ptr(), _ptr(q_w), _ptr(k_w), _ptr(rope), T, heads, kv_heads, head_dim, v_dim, int(planes), _ptr(q_scale),
+        positions.data_ptr(), _ptr(q_w), _ptr(k_w), _ptr(rope), T, heads, kv_heads, head_dim, v_dim, int(planes), _ptr(q_scale), _ptr(bias),
         page_size, float(eps), 1 if write_kv else 0, _code(qkv), _stream()))
 
 

@@ -288,10 +288,12 @@ class AttentionMixer(Mixer):
                              positions=step.positions, q_w=self.q_norm, k_w=self.k_norm, rope=rope, heads=s.heads,
                              kv_heads=s.kv_heads, head_dim=D, page_size=step.page_size, eps=self.qk_eps)
         else:
-            proj = rt.linear(x, w_in, "attn_qkv", b_in)
+            # (the vendor's product has no float32 bias: with many rows the kernel behind it adds the biases)
+            late = b_in if b_in is not None and rt.mode == "bfloat16" and rt.many_rows == "auto" and not rt.few_rows(x, w_in) else None
+            proj = rt.linear(x, w_in, "attn_qkv", None if late is not None else b_in)
             ops.qk_norm_rope_store(proj, q, cache.storage, table, step.seq_of_token, step.positions, self.q_norm,
                                    self.k_norm, rope, s.heads, s.kv_heads, D, step.page_size, self.qk_eps,
-                                   write_kv=cache.owner, v_dim=DV, planes=self.planes, q_scale=self.q_scale)
+                                   write_kv=cache.owner, v_dim=DV, planes=self.planes, q_scale=self.q_scale, bias=late)
         o = rt.ws.get("attn_o", (T, s.heads, DV), rt.act_dtype)
         gate = proj[:, gate_at:] if s.head_gate or s.out_gate else None
         self.attend(q, cache, table, step, gate, o)

@@ -119,8 +119,9 @@ class RoutedExperts(FeedForward):
         return out
 
     def __init__(self, spec, weights: Dict[str, torch.Tensor], rt):
-        if spec.top > 16:
-            raise ValueError(f"routed experts: top {spec.top} (at most 16 are supported)")
+        most = 16 if spec.score == "softmax" else 32
+        if spec.top > most:
+            raise ValueError(f"routed experts: top {spec.top} (at most {most} are supported)")
         if spec.score not in ("softmax", "sigmoid", "softmax_all") or spec.activation not in ("gated", "relu_squared"):
             raise ValueError(f"routed experts: score '{spec.score}' (softmax, sigmoid, softmax_all), activation '{spec.activation}' (gated, relu_squared)")
         self.identity = int(getattr(spec, "identity", 0))
