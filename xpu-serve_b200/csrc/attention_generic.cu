@@ -106,7 +106,7 @@ __global__ void qk_norm_rope_store_kernel(const T* __restrict__ qkv, int64_t ld,
 // bfloat16, head sizes 16, 32, 48, 64, 96, 128, 256: a thread owns 8 neighbouring channels (one 16-byte load and
 // store), the D / 8 threads of a head are neighbours in a warp (a warp holds as many whole heads as fit); the sum of
 // squares and the partner channels (i and i + D / 2 sit D / 16 lanes apart) travel by shuffles.
-template <int D>
+template <int D, bool BIAS>
 __global__ void __launch_bounds__(256) qk_norm_rope_store_vec_kernel(
     const __nv_bfloat16* __restrict__ qkv, int64_t ld, __nv_bfloat16* __restrict__ q_out, __nv_bfloat16* __restrict__ pool,
     const int32_t* __restrict__ page_table, int P, const int32_t* __restrict__ seq_of_token,
@@ -164,10 +164,8 @@ __global__ void __launch_bounds__(256) qk_norm_rope_store_vec_kernel(
         wv[4] = w1.x; wv[5] = w1.y; wv[6] = w1.z; wv[7] = w1.w;
     }
     const bool low = c0 < half;
-    float bv[8];
-#pragma unroll
-    for (int j = 0; j < 8; ++j) bv[j] = 0.0f;
-    if (bias != nullptr && live) {
+    float bv[8] = {0.0f, 0.0f, 0.0f, 0.0f, 0.0f, 0.0f, 0.0f, 0.0f};
+    if (BIAS && live) {
         const float4 b0 = *reinterpret_cast<const float4*>(bias + hh * D + c0), b1 = *reinterpret_cast<const float4*>(bias + hh * D + c0 + 4);
         bv[0] = b0.x; bv[1] = b0.y; bv[2] = b0.z; bv[3] = b0.w;
         bv[4] = b1.x; bv[5] = b1.y; bv[6] = b1.z; bv[7] = b1.w;
@@ -187,8 +185,8 @@ __global__ void __launch_bounds__(256) qk_norm_rope_store_vec_kernel(
 #pragma unroll
         for (int j = 0; j < 4; ++j) {
             const float2 f = __bfloat1622float2(h2[j]);
-            x[2 * j] = f.x + bv[2 * j];
-            x[2 * j + 1] = f.y + bv[2 * j + 1];
+            x[2 * j] = BIAS ? f.x + bv[2 * j] : f.x;
+            x[2 * j + 1] = BIAS ? f.y + bv[2 * j + 1] : f.y;
         }
     }
     float ss = 0.0f;
@@ -224,7 +222,7 @@ __global__ void __launch_bounds__(256) qk_norm_rope_store_vec_kernel(
         }
     }
     if (!live) return;
-    if (rotate || bias != nullptr) {
+    if (rotate || BIAS) {
         uint4 o;
         __nv_bfloat162* h2 = reinterpret_cast<__nv_bfloat162*>(&o);
 #pragma unroll
@@ -345,7 +343,7 @@ XS_API int xs_qk_norm_rope_store(const void* qkv, int64_t ld, void* q_out, void*
         const int64_t vitems = (int64_t)T * (Hq + (write_kv ? Hkv : 0) + (write_kv && planes > 1 ? ceil_div_i((int64_t)Hkv * DV, D) : 0));
         const int vblocks = ceil_div_i(ceil_div_i(vitems, 32 / (D / 8)), 8);       // 8 warps a block
 #define XS_ROPE_VEC(DD)                                                                                            \
-    xs_launch(qk_norm_rope_store_vec_kernel<DD>, dim3(vblocks), dim3(256), 0, stream, (const __nv_bfloat16*)qkv, ld, \
+    xs_launch(bias != nullptr ? qk_norm_rope_store_vec_kernel<DD, true> : qk_norm_rope_store_vec_kernel<DD, false>, dim3(vblocks), dim3(256), 0, stream, (const __nv_bfloat16*)qkv, ld, \
               (__nv_bfloat16*)q_out, (__nv_bfloat16*)pool, page_table, P, seq_of_token, positions, q_w, k_w,        \
               (const float2*)rope, T, Hq, Hkv, DV, planes, q_scale, bias, page_size, eps, write_kv)
         switch (D) {
