@@ -290,7 +290,7 @@ def dev_i32(v):
 
 
 ATTENTION_SHAPES = [   # H, G, D, DV, planes
-    (4, 2, 64, 64, 2), (4, 2, 64, 64, 1), (8, 1, 128, 32, 2), (4, 4, 48, 128, 2), (3, 1, 96, 64, 2), (6, 2, 16, 32, 2), (2, 2, 32, 32, 1),
+    (4, 2, 64, 64, 2), (4, 2, 64, 64, 1), (8, 2, 128, 32, 2), (4, 4, 48, 128, 2), (3, 1, 96, 64, 2), (6, 2, 16, 32, 2), (2, 2, 32, 32, 1),
     (20, 1, 64, 32, 2), (2, 1, 160, 72, 2), (2, 1, 128, 128, 1)]
 
 
@@ -401,7 +401,7 @@ def test_attention_kernels(kernel, shape, window, keep, plus_one, gated):
 
 
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
-@pytest.mark.parametrize("H,G,D,DV,planes", [(4, 2, 16, 32, 2), (8, 1, 128, 32, 2), (3, 3, 48, 64, 2), (2, 2, 64, 64, 1), (5, 1, 64, 128, 2), (2, 1, 6, 10, 2),
+@pytest.mark.parametrize("H,G,D,DV,planes", [(4, 2, 16, 32, 2), (8, 2, 128, 32, 2), (3, 3, 48, 32, 2), (2, 2, 64, 64, 1), (5, 1, 64, 128, 2), (2, 1, 6, 10, 2),
                                              (2, 2, 32, 48, 2), (1, 1, 256, 8, 2)])
 @pytest.mark.parametrize("biased", [False, True])
 def test_norm_rotation_and_store(biased, H, G, D, DV, planes, dtype):
@@ -474,7 +474,7 @@ def test_poly_norm_alone(F, dtype):
     assert (gap <= tol).all(), gap
 
 
-@pytest.mark.parametrize("E,identity,top,groups,keep", [(5, 1, 2, 2, 1), (16, 2, 4, 2, 1), (7, 2, 3, 3, 2), (8, 0, 1, 1, 1), (40, 24, 6, 8, 3), (60, 4, 8, 4, 4), (200, 56, 16, 16, 2), (60, 4, 29, 2, 1)])
+@pytest.mark.parametrize("E,identity,top,groups,keep", [(5, 1, 2, 2, 1), (14, 4, 5, 3, 2), (7, 2, 3, 3, 2), (8, 0, 1, 1, 1), (40, 24, 6, 8, 3), (60, 4, 8, 4, 4), (200, 56, 16, 16, 2), (60, 4, 29, 2, 1)])
 def test_routing_kernel_alone(E, identity, top, groups, keep):
     """Choices and weights against the oracle's wherever the choice is no close call; corrections of both signs, so that open
     groups hold negative choice scores."""
