@@ -104,7 +104,7 @@ def test_vl_wrapper_reads_text_config():
 def test_registry_dispatch_and_listing():
     assert registry.architecture_for({"model_type": "lfm3"}).config_class is Lfm3Config
     assert registry.architecture_for({"architectures": ["Lfm3ForCausalLM"]}).name == "lfm3"
-    with pytest.raises(ConfigError, match=r"'llama'.*supported: gararax, lfm3"):
+    with pytest.raises(ConfigError, match=r"'llama'.*supported: gararax, lazovik, lfm3"):
         registry.architecture_for({"model_type": "llama"})
 
 

@@ -6,8 +6,9 @@ from .nimelorn import NimelornConfig
 from .tozarax import TozaraxConfig
 from .vekuzen import VekuzenConfig
 from .gararax import GararaxConfig
+from .lazovik import LazovikConfig
 from .spec import (AttentionSpec, LayerCall, LayerSpec, ModelSpec, NormSpec, RopeSpec,
                    ShortConvSpec, SwiGLUSpec)
 
-__all__ = ["ConfigError", "read_json", "Lfm3Config", "Lfm3Rope", "SaralixConfig", "NimelornConfig", "TozaraxConfig", "VekuzenConfig", "GararaxConfig", "AttentionSpec", "LayerCall",
+__all__ = ["ConfigError", "read_json", "Lfm3Config", "Lfm3Rope", "SaralixConfig", "NimelornConfig", "TozaraxConfig", "VekuzenConfig", "GararaxConfig", "LazovikConfig", "AttentionSpec", "LayerCall",
            "LayerSpec", "ModelSpec", "NormSpec", "RopeSpec", "ShortConvSpec", "SwiGLUSpec"]

@@ -53,7 +53,8 @@ class AttentionSpec:
         "gate": "self_attn.gate_proj.weight",
         "q_norm": "self_attn.q_norm.weight", "k_norm": "self_attn.k_norm.weight",
         "q_bias": "self_attn.q_proj.bias", "k_bias": "self_attn.k_proj.bias", "v_bias": "self_attn.v_proj.bias",
-        "temp": "self_attn.temp"})
+        "temp": "self_attn.temp", "q_conv": "self_attn.q_conv.weight", "k_conv": "self_attn.k_conv.weight",
+        "v_conv": "self_attn.v_conv.weight", "o_bias": "self_attn.o_proj.bias"})
     kind: str = "attention"
     qkv_bias: bool = False   # q, k and v projections with a bias each (LFM3 has none)
     v_dim: int = 0           # size of a value head when it differs from head_dim (0: head_dim); needs position None, or v_layout "own"
@@ -68,6 +69,12 @@ class AttentionSpec:
     plus_one: bool = False   # softmax weights exp(s_j) / (1 + sum exp(s_j))
     out_gate: bool = False   # every channel of the concatenated heads times sigmoid((x Wg^T)[t, c]) (names["gate"])
     head_temp: bool = False  # scores of head h times a learned number (names["temp"])
+    qkv_taps: int = 0        # n > 0: q, k and v (biases included) each pass a causal filter of n taps per channel over the
+                             # sequence's tokens (names "q_conv", "k_conv", "v_conv": [channels, n]) before norm and rotation; the
+                             # last n - 1 rows of the projections are part of a sequence's state
+    qk_norm_all: bool = False  # RMSNorm over all of q (and all of k) at once, weights of those sizes, before the rotation (qk_norm_eps)
+    softcap: float = 0.0     # c > 0: a score is c tanh(score / c), before the mask and the softmax
+    o_bias: bool = False     # the output projection has a bias (names["o_bias"])
 
 
 @dataclass(frozen=True)
@@ -307,6 +314,7 @@ class RoutedExpertsSpec:
     renorm_eps: float = 0.0
     shared_gated: bool = True
     activation: str = "gated"        # "gated" (SwiGLU, or the clamped unit with `limit`) | "relu_squared"
+    weight_on: str = "output"        # "input": a choice's weight multiplies the expert's input instead of its output
 
 
 @dataclass(frozen=True)
@@ -343,6 +351,52 @@ class ParallelMixerSpec:
     scale: float
     eps: float
     kind: str = "parallel"
+
+
+@dataclass(frozen=True)
+class SummedMixerSpec:
+    """Mixers side by side that read the same input: the result is the sum of their outputs, branch k's times scales[k], with no
+    norm between. The branches' output projections run as one product over their heads side by side."""
+    hidden: int
+    branches: Tuple[object, ...]
+    scales: Tuple[float, ...]
+    kind: str = "parallel_sum"
+
+
+@dataclass(frozen=True)
+class TimeMixingSpec:
+    """RWKV-style time mixing: a memory [dim, dim] per head (float32) whose rows decay by exp(-exp(W2 tanh(W1 x_w) + w0)), read before
+    a token's own write with a bonus u on the token's own pair. r, k, v, the gate and the decay's hidden vector each read a mix of
+    their own of the token's input with the one before it (names "mu_r" to "mu_w"; the last input is part of a sequence's state).
+    The heads' outputs are divided by their root mean square (`eps`), multiplied by a weight over all heads and by silu of the
+    gate, then projected (parts/decay_memory.py)."""
+    hidden: int
+    heads: int
+    dim: int
+    rank: int                # rows of W1
+    eps: float
+    names: Dict[str, str] = field(default_factory=lambda: {
+        "mu_r": "mix.mu.r", "mu_k": "mix.mu.k", "mu_v": "mix.mu.v", "mu_g": "mix.mu.g", "mu_w": "mix.mu.w", "r": "mix.r", "k": "mix.k",
+        "v": "mix.v", "gate": "mix.g", "w1": "mix.w1", "w2": "mix.w2", "w0": "mix.w0", "u": "mix.u", "norm": "mix.norm", "o": "mix.o"})
+    kind: str = "time_mixing"
+
+
+@dataclass(frozen=True)
+class GatedLinearSpec:
+    """Gated linear attention: a memory [dim, vdim] per head (float32) whose rows decay by sigmoid(W2 (W1 x) + b)^(1 / tau), read behind
+    a token's own write with its query times dim^(-1/2). The heads' outputs are divided by their root mean square (`eps`),
+    multiplied by a weight of vdim entries that the heads share and by silu of a gate, then projected (parts/decay_memory.py)."""
+    hidden: int
+    heads: int
+    dim: int
+    vdim: int
+    rank: int                # rows of W1
+    tau: float
+    eps: float
+    names: Dict[str, str] = field(default_factory=lambda: {
+        "q": "mix.q", "k": "mix.k", "v": "mix.v", "gate": "mix.g", "a1": "mix.a1", "a2": "mix.a2", "a2_bias": "mix.a2.b", "norm": "mix.norm",
+        "o": "mix.o"})
+    kind: str = "gla"
 
 
 @dataclass(frozen=True)

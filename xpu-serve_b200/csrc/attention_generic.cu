@@ -241,8 +241,8 @@ __global__ void attention_generic_kernel(const T* __restrict__ q, const T* __res
                                          const int32_t* __restrict__ page_table, int P,
                                          const int32_t* __restrict__ seq_of_token,
                                          const int32_t* __restrict__ positions, const T* __restrict__ gate,
-                                         int64_t ld_gate, T* __restrict__ out, int Tn, int Hq, int Hkv, int D, int DV,
-                                         int planes, int page_size, float scale, int window, int keep, int plus_one,
+                                         int64_t ld_gate, T* __restrict__ out, int64_t ld_out, int Tn, int Hq, int Hkv, int D, int DV,
+                                         int planes, int page_size, float scale, float softcap, int window, int keep, int plus_one,
                                          int gate_channels) {
     extern __shared__ float q_sm[];   // [warps][D]
     pdl_launch_dependents();
@@ -279,7 +279,7 @@ __global__ void attention_generic_kernel(const T* __restrict__ q, const T* __res
                 const T* kr = pool + table[j / page_size] * page_elems + k_at + (int64_t)(j % page_size) * D;
                 float dot = 0.0f;
                 for (int d = 0; d < D; ++d) dot = fmaf(qs[d], to_f32(kr[d]), dot);
-                s = dot;
+                s = softcap > 0.0f ? softcap * tanhf(dot / softcap) : dot;
             }
             const float m_new = fmaxf(m, warp_max(s));
             const float p = j < end ? expf(s - m_new) : 0.0f;
@@ -307,7 +307,7 @@ __global__ void attention_generic_kernel(const T* __restrict__ q, const T* __res
         g = 1.0f / (1.0f + expf(-z));
     }
     const float norm = g / l;
-    T* orow = out + ((int64_t)t * Hq + h) * DV;
+    T* orow = out + (int64_t)t * ld_out + (int64_t)h * DV;
 #pragma unroll
     for (int u = 0; u < kMaxHeadDim / 32; ++u) {
         const int d = lane + 32 * u;
@@ -370,13 +370,14 @@ XS_API int xs_qk_norm_rope_store(const void* qkv, int64_t ld, void* q_out, void*
 
 XS_API int xs_attention_generic(const void* q, const void* pool, const int32_t* page_table, int P,
                                 const int32_t* seq_of_token, const int32_t* positions, const void* gate,
-                                int64_t ld_gate, void* out, int T, int Hq, int Hkv, int D, int DV, int planes, int page_size,
-                                float scale, int window, int keep, int plus_one, int gate_channels, int dtype,
+                                int64_t ld_gate, void* out, int64_t ld_out, int T, int Hq, int Hkv, int D, int DV, int planes, int page_size,
+                                float scale, float softcap, int window, int keep, int plus_one, int gate_channels, int dtype,
                                 cudaStream_t stream) {
     if (T == 0) return 0;
     XS_REQUIRE(D > 0 && D % 2 == 0 && D <= kMaxHeadDim, "attention: head size %d (even, at most %d)", D, kMaxHeadDim);
     XS_REQUIRE(DV > 0 && DV <= kMaxHeadDim && (planes == 2 || (planes == 1 && DV == D)), "attention: value size %d, %d planes", DV, planes);
     XS_REQUIRE(Hq > 0 && Hkv > 0 && Hq % Hkv == 0, "attention: %d heads over %d kv heads", Hq, Hkv);
+    XS_REQUIRE(softcap >= 0.0f && ld_out >= (int64_t)Hq * DV, "attention: soft cap %g, output rows %lld apart", (double)softcap, (long long)ld_out);
     XS_REQUIRE(page_size > 0 && P > 0 && keep >= 0, "attention: window %d, page size %d, %d pages", window, page_size, P);
     const int warps = 4;
     const int blocks = ceil_div_i((int64_t)T * Hq, warps);
@@ -384,7 +385,7 @@ XS_API int xs_attention_generic(const void* q, const void* pool, const int32_t* 
     XS_DISPATCH_DTYPE(dtype, TT,
                       attention_generic_kernel<TT><<<blocks, warps * 32, smem, stream>>>(
                           (const TT*)q, (const TT*)pool, page_table, P, seq_of_token, positions, (const TT*)gate,
-                          ld_gate, (TT*)out, T, Hq, Hkv, D, DV, planes, page_size, scale, window, keep, plus_one, gate_channels));
+                          ld_gate, (TT*)out, ld_out, T, Hq, Hkv, D, DV, planes, page_size, scale, softcap, window, keep, plus_one, gate_channels));
     XS_LAUNCH_CHECK("attention_generic");
     return 0;
 }

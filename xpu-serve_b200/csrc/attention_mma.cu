@@ -198,6 +198,8 @@ __global__ void __launch_bounds__(160) attention_decode_tma_kernel(const __grid_
             mma_bf16(sc[0], qf[kk], b0, b1);
             mma_bf16(sc[1], qf[kk], b2, b3);
         }
+        const float to_log2 = p.cap_out > 0.0f ? 1.0f : p.scale_log2;
+        if (p.cap_out > 0.0f) xs_cap_scores<8>(&sc[0][0], p.cap_in, p.cap_out);
         const int key0 = b * BN + warp * 16 + (lane & 3) * 2;
         float mx1 = -INFINITY, mx2 = -INFINITY;
 #pragma unroll
@@ -207,8 +209,8 @@ __global__ void __launch_bounds__(160) attention_decode_tma_kernel(const __grid_
                 const int key = key0 + i * 8 + e;
                 const bool v1 = key <= pos1 && (key >= lo1 || key < p.keep);
                 const bool v2 = key <= pos2 && (key >= lo2 || key < p.keep);
-                sc[i][e] = v1 ? sc[i][e] * p.scale_log2 : -INFINITY;
-                sc[i][2 + e] = v2 ? sc[i][2 + e] * p.scale_log2 : -INFINITY;
+                sc[i][e] = v1 ? sc[i][e] * to_log2 : -INFINITY;
+                sc[i][2 + e] = v2 ? sc[i][2 + e] * to_log2 : -INFINITY;
                 mx1 = fmaxf(mx1, sc[i][e]);
                 mx2 = fmaxf(mx2, sc[i][2 + e]);
             }
@@ -295,7 +297,7 @@ __global__ void __launch_bounds__(160) attention_decode_tma_kernel(const __grid_
         if (p.splits == 1) {
             float f = inv_denominator(l, m, p.plus_one);
             if (p.gate != nullptr) f *= gate_of(p, t, p.gate_channels ? h * D + d : h);
-            p.out[row * D + d] = __float2bfloat16_rn(acc * f);
+            p.out[(int64_t)t * p.ld_out + h * D + d] = __float2bfloat16_rn(acc * f);
         } else {
             p.part_o[(row * p.splits + split) * D + d] = acc;
             if (d == 0) {
@@ -352,7 +354,7 @@ __global__ void __launch_bounds__(160) attention_decode_tma_kernel(const __grid_
             f0 *= gate_of(p, t, h * D + d);
             f1 *= gate_of(p, t, h * D + d + 1);
         }
-        *reinterpret_cast<__nv_bfloat162*>(p.out + row * D + d) = __floats2bfloat162_rn(a0 * f0, a1 * f1);
+        *reinterpret_cast<__nv_bfloat162*>(p.out + (int64_t)t * p.ld_out + h * D + d) = __floats2bfloat162_rn(a0 * f0, a1 * f1);
     }
     if (threadIdx.x == 0) *counter = 0;
 }
@@ -361,7 +363,7 @@ __global__ void __launch_bounds__(160) attention_decode_tma_kernel(const __grid_
 // splits s and s + 32's (max, sum) and weights (splits <= 64), and the partial outputs are read with independent loads.
 __global__ void attention_combine_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml,
                                          const __nv_bfloat16* __restrict__ gate, int64_t ld_gate,
-                                         __nv_bfloat16* __restrict__ out, int64_t rows, int Hq, int D, int splits,
+                                         __nv_bfloat16* __restrict__ out, int64_t ld_out, int64_t rows, int Hq, int D, int splits,
                                          int plus_one, int gate_channels) {
     pdl_launch_dependents();
     pdl_wait();
@@ -404,7 +406,7 @@ __global__ void attention_combine_kernel(const float* __restrict__ part_o, const
                 f0 *= 1.0f / (1.0f + __expf(-__bfloat162float(gate_row[d])));
                 f1 *= 1.0f / (1.0f + __expf(-__bfloat162float(gate_row[d + 1])));
             }
-            *reinterpret_cast<__nv_bfloat162*>(out + row * D + d) = __floats2bfloat162_rn(a0 * f0, a1 * f1);
+            *reinterpret_cast<__nv_bfloat162*>(out + (row / Hq) * ld_out + (row % Hq) * D + d) = __floats2bfloat162_rn(a0 * f0, a1 * f1);
         }
     }
 }
@@ -539,9 +541,9 @@ XS_API void xs_attention_mma_set_tma_carveout(int percent) { g_attn_tma_carveout
 // non-zero when a wait gave up (the result is then invalid); with them, decoding at head size 64 takes the TMA-fed kernel.
 XS_API int xs_attention_mma_merged(const void* q, const void* pool, const int32_t* page_table, int P,
                                    const int32_t* cu_seqlens, const int32_t* kv_lens, const void* gate, int64_t ld_gate,
-                                   void* out, void* scratch, int64_t scratch_bytes, void* counters, int64_t pool_pages,
+                                   void* out, int64_t ld_out, void* scratch, int64_t scratch_bytes, void* counters, int64_t pool_pages,
                                    int* status, int T, int n_seqs, int max_q_len, int Hq, int Hkv, int D, int DV, int planes,
-                                   int page_size, float scale, int window, int keep, int plus_one, int gate_channels, int splits,
+                                   int page_size, float scale, float softcap, int window, int keep, int plus_one, int gate_channels, int splits,
                                    cudaStream_t stream) {
     if (T == 0) return 0;
     XS_REQUIRE(Hq > 0 && Hkv > 0 && Hq % Hkv == 0, "attention: %d heads over %d kv heads", Hq, Hkv);
@@ -554,6 +556,7 @@ XS_API int xs_attention_mma_merged(const void* q, const void* pool, const int32_
                "attention: bad sizes (1 to 64 key splits)");
     XS_REQUIRE(n_seqs <= 65535 && (int64_t)Hkv * splits <= 65535, "attention: grid too large");
     const int64_t need = xs_attention_mma_scratch_bytes((int64_t)T * Hq, DV, splits);
+    XS_REQUIRE(softcap >= 0.0f && ld_out >= (int64_t)Hq * DV && ld_out % 2 == 0, "attention: soft cap %g, output rows %lld apart", (double)softcap, (long long)ld_out);
     XS_REQUIRE((uintptr_t)out % 4 == 0 && (splits == 1 || (uintptr_t)scratch % 16 == 0), "attention: out or scratch is misaligned");
     XS_REQUIRE(splits == 1 || (scratch != nullptr && scratch_bytes >= need),
                "attention: %lld bytes of scratch needed for %d splits, %lld given", (long long)need, splits,
@@ -568,6 +571,7 @@ XS_API int xs_attention_mma_merged(const void* q, const void* pool, const int32_
     p.gate = (const __nv_bfloat16*)gate;
     p.ld_gate = ld_gate;
     p.out = (__nv_bfloat16*)out;
+    p.ld_out = ld_out;
     p.part_o = (float*)scratch;
     p.part_ml = p.part_o + (int64_t)T * Hq * splits * DV;
     p.Hq = Hq;
@@ -583,6 +587,8 @@ XS_API int xs_attention_mma_merged(const void* q, const void* pool, const int32_
     p.splits = splits;
     p.prefetch_blocks = g_attn_prefetch_blocks;
     p.scale_log2 = scale * 1.4426950408889634f;
+    p.cap_in = softcap > 0.0f ? scale / softcap : 0.0f;
+    p.cap_out = softcap > 0.0f ? softcap * 1.4426950408889634f : 0.0f;
     p.counters = (p.decode_rows && splits > 1) ? (unsigned int*)counters : nullptr;
     const int max_tiles = ceil_div_i(max_q_len, p.tokens_per_tile);
     if (D != DV) {
@@ -612,7 +618,7 @@ XS_API int xs_attention_mma_merged(const void* q, const void* pool, const int32_
     if (splits > 1 && p.counters == nullptr) {
         const int64_t rows = (int64_t)T * Hq;
         xs_launch(attention_combine_kernel, dim3(ceil_div_i(rows, 4)), dim3(128), 0, stream, (const float*)p.part_o,
-                  (const float*)p.part_ml, p.gate, ld_gate, p.out, rows, Hq, DV, splits, p.plus_one, p.gate_channels);
+                  (const float*)p.part_ml, p.gate, ld_gate, p.out, ld_out, rows, Hq, DV, splits, p.plus_one, p.gate_channels);
         XS_LAUNCH_CHECK("attention_combine");
     }
     return 0;
@@ -622,8 +628,8 @@ XS_API int xs_attention_mma(const void* q, const void* pool, const int32_t* page
                             const int32_t* cu_seqlens, const int32_t* kv_lens, const void* gate, int64_t ld_gate,
                             void* out, void* scratch, int64_t scratch_bytes, int T, int n_seqs, int max_q_len, int Hq,
                             int Hkv, int D, int page_size, float scale, int window, int splits, cudaStream_t stream) {
-    return xs_attention_mma_merged(q, pool, page_table, P, cu_seqlens, kv_lens, gate, ld_gate, out, scratch, scratch_bytes,
-                                   nullptr, 0, nullptr, T, n_seqs, max_q_len, Hq, Hkv, D, D, 2, page_size, scale, window, 0, 0, 0,
+    return xs_attention_mma_merged(q, pool, page_table, P, cu_seqlens, kv_lens, gate, ld_gate, out, (int64_t)Hq * D, scratch, scratch_bytes,
+                                   nullptr, 0, nullptr, T, n_seqs, max_q_len, Hq, Hkv, D, D, 2, page_size, scale, 0.0f, window, 0, 0, 0,
                                    splits, stream);
 }
 

@@ -26,7 +26,8 @@ struct AttnParams {
     const int32_t* kv_lens;          // [n_seqs] length after this step
     const __nv_bfloat16* gate;       // [T, ld_gate] gate logits (one a head, or with gate_channels one a channel) or null
     int64_t ld_gate;
-    __nv_bfloat16* out;              // [T, Hq, DV]
+    __nv_bfloat16* out;              // [T, Hq, DV], tokens `ld_out` elements apart
+    int64_t ld_out;
     float* part_o;                   // [T * Hq, splits, DV]
     float* part_ml;                  // [T * Hq, splits, 2]
     int Hq, Hkv, G, tokens_per_tile, window, splits;
@@ -37,6 +38,7 @@ struct AttnParams {
     int prefetch_blocks;             // decode: how many of a CTA's first key blocks are hinted into L2 before the wait
     int decode_rows;                 // every tile has at most 16 rows: the warps split the keys instead
     float scale_log2;
+    float cap_in, cap_out;           // cap_out > 0: a score is cap_out * tanh(q.k * cap_in) (base-2 units) instead of q.k * scale_log2
     unsigned int* counters;          // decode with key splits: one zeroed word per (sequence, kv head), left zeroed; or null
 };
 
@@ -212,6 +214,8 @@ __global__ void __launch_bounds__(NTHREADS, prompt_ctas(D, DV)) attention_mma_ke
                     mma_bf16(s[2 * np + 1], qf[kk], b2, b3);
                 }
             }
+            const float to_log2 = p.cap_out > 0.0f ? 1.0f : p.scale_log2;
+            if (p.cap_out > 0.0f) xs_cap_scores<BN / 2>(&s[0][0], p.cap_in, p.cap_out);
             // scale, mask, running max. A block that every row of the tile sees whole (all of it at or before
             // the tile's first position and inside every row's window) needs no per-element test.
             const int key0 = b * BN + (lane & 3) * 2;
@@ -222,8 +226,8 @@ __global__ void __launch_bounds__(NTHREADS, prompt_ctas(D, DV)) attention_mma_ke
                 for (int i = 0; i < BN / 8; ++i) {
 #pragma unroll
                     for (int e = 0; e < 2; ++e) {
-                        s[i][e] = pos1 >= 0 ? s[i][e] * p.scale_log2 : -INFINITY;
-                        s[i][2 + e] = pos2 >= 0 ? s[i][2 + e] * p.scale_log2 : -INFINITY;
+                        s[i][e] = pos1 >= 0 ? s[i][e] * to_log2 : -INFINITY;
+                        s[i][2 + e] = pos2 >= 0 ? s[i][2 + e] * to_log2 : -INFINITY;
                         mx1 = fmaxf(mx1, s[i][e]);
                         mx2 = fmaxf(mx2, s[i][2 + e]);
                     }
@@ -236,8 +240,8 @@ __global__ void __launch_bounds__(NTHREADS, prompt_ctas(D, DV)) attention_mma_ke
                         const int key = key0 + i * 8 + e;
                         const bool v1 = key <= pos1 && (key >= lo1 || key < p.keep);
                         const bool v2 = key <= pos2 && (key >= lo2 || key < p.keep);
-                        s[i][e] = v1 ? s[i][e] * p.scale_log2 : -INFINITY;
-                        s[i][2 + e] = v2 ? s[i][2 + e] * p.scale_log2 : -INFINITY;
+                        s[i][e] = v1 ? s[i][e] * to_log2 : -INFINITY;
+                        s[i][2 + e] = v2 ? s[i][2 + e] * to_log2 : -INFINITY;
                         mx1 = fmaxf(mx1, s[i][e]);
                         mx2 = fmaxf(mx2, s[i][2 + e]);
                     }
@@ -302,7 +306,7 @@ __global__ void __launch_bounds__(NTHREADS, prompt_ctas(D, DV)) attention_mma_ke
         if (p.splits == 1) {
             float f = inv_denominator(l, m, p.plus_one);
             if (p.gate != nullptr && !p.gate_channels) f *= gate_of(p, t, h);
-            __nv_bfloat16* dst = p.out + row * DV + (lane & 3) * 2;
+            __nv_bfloat16* dst = p.out + (int64_t)t * p.ld_out + h * DV + (lane & 3) * 2;
             __nv_bfloat162 gates[DTILES];        // (all asked for before the first is used)
             if (p.gate_channels) {
                 const __nv_bfloat16* from = p.gate + (int64_t)t * p.ld_gate + h * DV + (lane & 3) * 2;
@@ -463,6 +467,8 @@ __global__ void __launch_bounds__(NTHREADS) attention_decode_mma_kernel(const At
             mma_bf16(s[0], qf[kk], b0, b1);
             mma_bf16(s[1], qf[kk], b2, b3);
         }
+        const float to_log2 = p.cap_out > 0.0f ? 1.0f : p.scale_log2;
+        if (p.cap_out > 0.0f) xs_cap_scores<8>(&s[0][0], p.cap_in, p.cap_out);
         const int key0 = b * BN + warp * 16 + (lane & 3) * 2;
         float mx1 = -INFINITY, mx2 = -INFINITY;
 #pragma unroll
@@ -472,8 +478,8 @@ __global__ void __launch_bounds__(NTHREADS) attention_decode_mma_kernel(const At
                 const int key = key0 + i * 8 + e;
                 const bool v1 = key <= pos1 && (key >= lo1 || key < p.keep);
                 const bool v2 = key <= pos2 && (key >= lo2 || key < p.keep);
-                s[i][e] = v1 ? s[i][e] * p.scale_log2 : -INFINITY;
-                s[i][2 + e] = v2 ? s[i][2 + e] * p.scale_log2 : -INFINITY;
+                s[i][e] = v1 ? s[i][e] * to_log2 : -INFINITY;
+                s[i][2 + e] = v2 ? s[i][2 + e] * to_log2 : -INFINITY;
                 mx1 = fmaxf(mx1, s[i][e]);
                 mx2 = fmaxf(mx2, s[i][2 + e]);
             }
@@ -554,7 +560,7 @@ __global__ void __launch_bounds__(NTHREADS) attention_decode_mma_kernel(const At
         if (p.splits == 1) {
             float f = inv_denominator(l, m, p.plus_one);
             if (p.gate != nullptr) f *= gate_of(p, t, p.gate_channels ? h * DV + d : h);
-            p.out[row * DV + d] = __float2bfloat16_rn(acc * f);
+            p.out[(int64_t)t * p.ld_out + h * DV + d] = __float2bfloat16_rn(acc * f);
         } else {
             p.part_o[(row * p.splits + split) * DV + d] = acc;
             if (d == 0) {
@@ -613,7 +619,7 @@ __global__ void __launch_bounds__(NTHREADS) attention_decode_mma_kernel(const At
             f0 *= gate_of(p, t, h * DV + d);
             f1 *= gate_of(p, t, h * DV + d + 1);
         }
-        *reinterpret_cast<__nv_bfloat162*>(p.out + row * DV + d) = __floats2bfloat162_rn(a0 * f0, a1 * f1);
+        *reinterpret_cast<__nv_bfloat162*>(p.out + (int64_t)t * p.ld_out + h * DV + d) = __floats2bfloat162_rn(a0 * f0, a1 * f1);
     }
     if (threadIdx.x == 0) *counter = 0;          // ready for the next call
 }

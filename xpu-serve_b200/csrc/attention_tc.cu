@@ -43,7 +43,8 @@ struct AttnTcParams {
     const int32_t* kv_lens;
     const __nv_bfloat16* gate;       // [T, ld_gate] or null
     int64_t ld_gate;
-    __nv_bfloat16* out;              // [T, Hq, D]
+    __nv_bfloat16* out;              // [T, Hq, D], tokens `ld_out` elements apart
+    int64_t ld_out;
     int* status;
     int Hq, Hkv, G, tokens_per_tile, window;
     int keep;                        // beside a window: the sequence's first positions that stay visible
@@ -51,6 +52,7 @@ struct AttnTcParams {
     int plus_one;                    // the softmax's denominator has one more term of score 0
     int gate_channels;               // gate logits per channel instead of per head
     float scale_log2;
+    float cap_in, cap_out;           // (CAP) a score is cap_out * tanh(q.k * cap_in), in base-2 units
     int order;
 };
 
@@ -114,7 +116,8 @@ __device__ __forceinline__ uint64_t smem_desc_sw128_mn(uint32_t addr) {
     return d;
 }
 
-template <int D>
+// CAP: scores pass a soft cap before the softmax (its own instance: the scores fill a thread's registers as it is).
+template <int D, bool CAP>
 __global__ void __launch_bounds__(kAttnThreads, 1)
 attention_tc_kernel(const __grid_constant__ CUtensorMap tmap_kv, const AttnTcParams p) {
     static_assert(D == 64, "one 128-byte swizzle atom a row");
@@ -320,6 +323,19 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap tmap_kv, const AttnTcPar
             for (int c = 0; c < TN; c += 32) tmem_ld32_nowait(lane_base + s_col + (uint32_t)c, raw + c);
             tmem_ld_wait();
             float mx4[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
+            if constexpr (CAP) {
+                // (columns that hold no key may hold anything here: they are replaced below)
+                float hi4 = 0.0f;
+#pragma unroll
+                for (int e = 0; e < TN; ++e) hi4 = fmaxf(hi4, fabsf(__uint_as_float(raw[e])));
+                if (__any_sync(0xffffffffu, hi4 * p.cap_in > kTanhNear)) {
+#pragma unroll
+                    for (int e = 0; e < TN; ++e) raw[e] = __float_as_uint(p.cap_out * xs_tanh(__uint_as_float(raw[e]) * p.cap_in));
+                } else {
+#pragma unroll
+                    for (int e = 0; e < TN; ++e) raw[e] = __float_as_uint(p.cap_out * xs_tanh_near(__uint_as_float(raw[e]) * p.cap_in));
+                }
+            }
             if (plain) {
 #pragma unroll
                 for (int e = 0; e < TN; ++e) mx4[e & 3] = fmaxf(mx4[e & 3], __uint_as_float(raw[e]));
@@ -333,7 +349,7 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap tmap_kv, const AttnTcPar
                 }
             }
             // the scale is positive: the largest scaled score is the scaled largest score
-            const float mx = fmaxf(fmaxf(mx4[0], mx4[1]), fmaxf(mx4[2], mx4[3])) * p.scale_log2;
+            const float mx = fmaxf(fmaxf(mx4[0], mx4[1]), fmaxf(mx4[2], mx4[3])) * (CAP ? 1.0f : p.scale_log2);
             const float m_new = fmaxf(m, mx);
             const float mb = m_new == -INFINITY ? 0.0f : m_new;
             const float alpha = ex2(m - mb);                      // 0 while nothing was seen
@@ -360,7 +376,7 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap tmap_kv, const AttnTcPar
                 float w[8];
 #pragma unroll
                 for (int e = 0; e < 8; ++e) {
-                    w[e] = ex2(fmaf(__uint_as_float(raw[8 * i + e]), p.scale_log2, -mb));   // ex2(-inf) = 0
+                    w[e] = ex2(CAP ? __uint_as_float(raw[8 * i + e]) - mb : fmaf(__uint_as_float(raw[8 * i + e]), p.scale_log2, -mb));   // ex2(-inf) = 0
                     add4[e & 3] += w[e];
                 }
                 *reinterpret_cast<uint4*>(p_row + (i >> 3) * (TM * 128) + (((i & 7) ^ (r & 7)) << 4)) =
@@ -427,7 +443,7 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap tmap_kv, const AttnTcPar
             float f = l > 0.0f ? 1.0f / l : 0.0f;
             if (p.gate != nullptr && !p.gate_channels) f *= 1.0f / (1.0f + __expf(-__bfloat162float(p.gate[(int64_t)t * p.ld_gate + h])));
             const float f0 = a0 * f, f1 = a1 * f;
-            uint4* dst = reinterpret_cast<uint4*>(p.out + ((int64_t)t * p.Hq + h) * D);
+            uint4* dst = reinterpret_cast<uint4*>(p.out + (int64_t)t * p.ld_out + h * D);
 #pragma unroll
             for (int c = 0; c < D / 8; ++c) {
                 float v[8];
@@ -465,8 +481,8 @@ XS_API int xs_attention_tc_supports(int D, int page_size, int G) {
 // status: one device int that the kernel sets non-zero if a wait inside it gave up (the result is then invalid).
 // max_kv_len: the longest sequence's keys, or 0 if the host does not know; it only picks the order in which CTAs start.
 XS_API int xs_attention_tc(const void* q, const void* pool, int64_t pool_pages, const int32_t* page_table, int P,
-                           const int32_t* cu_seqlens, const int32_t* kv_lens, const void* gate, int64_t ld_gate, void* out,
-                           int T, int n_seqs, int max_q_len, int Hq, int Hkv, int D, int planes, int page_size, float scale,
+                           const int32_t* cu_seqlens, const int32_t* kv_lens, const void* gate, int64_t ld_gate, void* out, int64_t ld_out,
+                           int T, int n_seqs, int max_q_len, int Hq, int Hkv, int D, int planes, int page_size, float scale, float softcap,
                            int window, int keep, int plus_one, int gate_channels, int max_kv_len, int* status,
                            cudaStream_t stream) {
     if (T == 0) return 0;
@@ -479,6 +495,7 @@ XS_API int xs_attention_tc(const void* q, const void* pool, int64_t pool_pages, 
     XS_REQUIRE(n_seqs <= 65535 && Hkv <= 65535, "attention (tcgen05): grid too large");
     XS_REQUIRE((uintptr_t)q % 16 == 0 && (uintptr_t)pool % 16 == 0 && (uintptr_t)out % 16 == 0,
                "attention (tcgen05): operands must be 16-byte aligned");
+    XS_REQUIRE(softcap >= 0.0f && ld_out >= (int64_t)Hq * D && ld_out % 8 == 0, "attention (tcgen05): soft cap %g, output rows %lld apart", (double)softcap, (long long)ld_out);
     XS_REQUIRE((planes == 1 || planes == 2) && keep >= 0 && scale > 0.0f, "attention (tcgen05): %d planes, %d kept, scale %g", planes, keep, (double)scale);
     XS_REQUIRE(gate == nullptr || !gate_channels || (ld_gate % 8 == 0 && (uintptr_t)gate % 16 == 0),
                "attention (tcgen05): a gate per channel needs 16-byte rows");
@@ -493,6 +510,7 @@ XS_API int xs_attention_tc(const void* q, const void* pool, int64_t pool_pages, 
     p.gate = (const __nv_bfloat16*)gate;
     p.ld_gate = ld_gate;
     p.out = (__nv_bfloat16*)out;
+    p.ld_out = ld_out;
     p.status = status;
     p.Hq = Hq;
     p.Hkv = Hkv;
@@ -504,19 +522,22 @@ XS_API int xs_attention_tc(const void* q, const void* pool, int64_t pool_pages, 
     p.plus_one = plus_one;
     p.gate_channels = gate != nullptr ? gate_channels : 0;
     p.scale_log2 = scale * 1.4426950408889634f;
+    p.cap_in = softcap > 0.0f ? scale / softcap : 0.0f;
+    p.cap_out = softcap > 0.0f ? softcap * 1.4426950408889634f : 0.0f;
     // All kv heads of the latest tiles first (5 to 15 % faster up to 8,192 keys: the long tiles of every head start
     // before any short one) while the keys and values of all heads together stay well inside L2; one head after the
     // other beyond that (1.5 % faster at 32,000 keys).
     p.order = max_kv_len <= 0 || (int64_t)max_kv_len * Hkv * D * 4 <= (int64_t)32 << 20;
     const int max_tiles = ceil_div_i(max_q_len, p.tokens_per_tile);
     const size_t smem = (size_t)TM * D * 2 + (size_t)KV_STAGES * 4 * PAGE * D * 2 + 2 * (size_t)TM * TN * 2 + 1024;
-    static bool opted = false;
-    if (!opted) {
-        cudaFuncSetAttribute(attention_tc_kernel<64>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-        opted = true;
+    static bool opted[2] = {};
+    const auto kernel = softcap > 0.0f ? attention_tc_kernel<64, true> : attention_tc_kernel<64, false>;
+    if (!opted[softcap > 0.0f]) {
+        cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        opted[softcap > 0.0f] = true;
     }
     const dim3 grid(max_tiles, n_seqs, Hkv);
-    XS_REQUIRE(xs_launch(attention_tc_kernel<64>, grid, dim3(kAttnThreads), smem, stream, map, p) == cudaSuccess,
+    XS_REQUIRE(xs_launch(kernel, grid, dim3(kAttnThreads), smem, stream, map, p) == cudaSuccess,
                "attention (tcgen05): launch failed: %s", cudaGetErrorString(cudaGetLastError()));
     return 0;
 }

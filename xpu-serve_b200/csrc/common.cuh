@@ -106,6 +106,38 @@ __device__ __forceinline__ XsBlocks xs_blocks(int pos0, int hi, int window, int 
     return b;
 }
 
+// tanh(x) to about 1e-7 absolute, by one hardware exponential and one division: 1 - 2 / (1 + e^(2x)) (saturates to 1 and -1).
+__device__ __forceinline__ float xs_tanh(float x) {
+    float e;
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(e) : "f"(x * 2.8853900817779268f));
+    return 1.0f - __fdividef(2.0f, 1.0f + e);
+}
+// The same for |x| <= kTanhNear by the first six terms of the Taylor series (the seventh is below 2e-9 of the result): no
+// hardware exponential, which is the scarce unit of a softmax.
+constexpr float kTanhNear = 0.3f;
+__device__ __forceinline__ float xs_tanh_near(float x) {
+    const float z = x * x;
+    float p = fmaf(z, -1382.0f / 155925.0f, 62.0f / 2835.0f);
+    p = fmaf(z, p, -17.0f / 315.0f);
+    p = fmaf(z, p, 2.0f / 15.0f);
+    p = fmaf(z, p, -1.0f / 3.0f);
+    return fmaf(x * z, p, x);
+}
+// n scores s in place: cap_out * tanh(s * cap_in), the series where the whole warp's allow it.
+template <int N>
+__device__ __forceinline__ void xs_cap_scores(float* s, float cap_in, float cap_out) {
+    float most = 0.0f;
+#pragma unroll
+    for (int i = 0; i < N; ++i) most = fmaxf(most, fabsf(s[i]));
+    if (__any_sync(0xffffffffu, most * cap_in > kTanhNear)) {
+#pragma unroll
+        for (int i = 0; i < N; ++i) s[i] = cap_out * xs_tanh(s[i] * cap_in);
+    } else {
+#pragma unroll
+        for (int i = 0; i < N; ++i) s[i] = cap_out * xs_tanh_near(s[i] * cap_in);
+    }
+}
+
 static inline int ceil_div_i(int64_t a, int64_t b) { return (int)((a + b - 1) / b); }
 
 // ---- programmatic dependent launch ------------------------------------------------------------

@@ -236,10 +236,11 @@ __global__ void moe_route_warp_kernel(const float* __restrict__ logits, int ld, 
 // with `renorm`.
 // `score` 1: s is the softmax over all E logits instead of their sigmoids. Experts from `real` on have no weights (their
 // output is their input): a choice of one is written as id -1, with its weight.
+// `squared`: the weights' squares are written (experts that are homogeneous of degree two, fed their weight times the input).
 // A warp per token; the token's s and c stand in shared memory (2 E floats a warp).
 __global__ void moe_route_grouped_kernel(const float* __restrict__ logits, int ld, int T, int E, int top,
                                          const float* __restrict__ correction, int groups, int keep, int group_top, float scale,
-                                         int renorm, float renorm_eps, int score, int real, int32_t* __restrict__ ids,
+                                         int renorm, float renorm_eps, int squared, int score, int real, int32_t* __restrict__ ids,
                                          float* __restrict__ wts) {
     extern __shared__ float route_smem[];
     pdl_launch_dependents();
@@ -333,7 +334,8 @@ __global__ void moe_route_grouped_kernel(const float* __restrict__ logits, int l
     }
     if (lane < top) {
         ids[(int64_t)t * top + lane] = mine_id < real ? mine_id : -1;        // (an expert without weights: its input passes)
-        wts[(int64_t)t * top + lane] = (renorm ? mine / (sum + renorm_eps) : mine) * scale;
+        const float w = (renorm ? mine / (sum + renorm_eps) : mine) * scale;
+        wts[(int64_t)t * top + lane] = squared ? w * w : w;
     }
 }
 
@@ -589,7 +591,7 @@ XS_API int xs_moe_route(const float* logits, int ld, int T, int E, int top, floa
 }
 
 XS_API int xs_moe_route_grouped(const float* logits, int ld, int T, int E, int top, const float* correction, int groups, int keep,
-                                int group_top, float scale, int renorm, float renorm_eps, int score, int real, int32_t* ids,
+                                int group_top, float scale, int renorm, float renorm_eps, int squared, int score, int real, int32_t* ids,
                                 float* wts, cudaStream_t stream) {
     if (T == 0) return 0;
     XS_REQUIRE(T > 0 && E > 0 && top > 0 && top <= E && top <= 32 && ld >= E,
@@ -603,7 +605,7 @@ XS_API int xs_moe_route_grouped(const float* logits, int ld, int T, int E, int t
     XS_REQUIRE(per_warp <= 40 * 1024, "moe_route_grouped: %d experts are more than the kernel's shared memory holds", E);
     const int warps = per_warp * 4 <= 40 * 1024 ? 4 : 1;
     xs_launch(moe_route_grouped_kernel, dim3(ceil_div_i(T, warps)), dim3(32 * warps), per_warp * warps, stream, logits, ld, T, E, top,
-              correction, groups, keep, group_top, scale, renorm, renorm_eps, score, real, ids, wts);
+              correction, groups, keep, group_top, scale, renorm, renorm_eps, squared, score, real, ids, wts);
     XS_LAUNCH_CHECK("moe_route_grouped");
     return 0;
 }

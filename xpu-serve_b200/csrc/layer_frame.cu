@@ -444,6 +444,17 @@ __global__ void stream_add_vec_kernel(float4* __restrict__ h, const float4* __re
 
 }  // namespace
 
+// A sequence's filter state alone: its last taps - 1 rows of x (of the step's rows, and the state's own where the step brought
+// fewer). For kernels that hold a filter of their own.
+int xs_filter_state(const void* x, int64_t ldx, void* state, const int32_t* cu_seqlens, const int32_t* slots, int n_seqs, int C,
+                    int taps, int dtype, cudaStream_t stream) {
+    XS_DISPATCH_DTYPE(dtype, TT,
+                      xs_launch(causal_conv_state_kernel<TT>, dim3(n_seqs, ceil_div_i(C, 128)), dim3(128), 0, stream, (const TT*)x, ldx,
+                                (TT*)state, cu_seqlens, slots, C, taps));
+    XS_LAUNCH_CHECK("causal_conv (state)");
+    return 0;
+}
+
 XS_API int xs_embed_pos(const void* table, const void* rows, int dtype, const int32_t* ids, const int32_t* positions, float* h,
                         int T, int H, float scale, cudaStream_t stream) {
     if (T == 0) return 0;
@@ -562,10 +573,7 @@ XS_API int xs_causal_conv(const void* x, int64_t ldx, const float* taps_w, void*
     }
     XS_LAUNCH_CHECK("causal_conv");
     if (taps > 1) {
-        XS_DISPATCH_DTYPE(dtype, TT,
-                          xs_launch(causal_conv_state_kernel<TT>, dim3(n_seqs, tiles), dim3(128), 0, stream, (const TT*)x, ldx,
-                                    (TT*)state, cu_seqlens, slots, C, taps));
-        XS_LAUNCH_CHECK("causal_conv (state)");
+        return xs_filter_state(x, ldx, state, cu_seqlens, slots, n_seqs, C, taps, dtype, stream);
     }
     return 0;
 }

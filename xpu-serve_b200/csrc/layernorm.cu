@@ -176,13 +176,14 @@ __global__ void add_layernorm_vec_kernel(float* __restrict__ h, const TM* __rest
 // gate_act 1 by silu(gate[t, g, :]) = gate * sigmoid(gate).
 template <typename TY>
 __global__ void grouped_rmsnorm_kernel(const float* __restrict__ x, const float* __restrict__ w, TY* __restrict__ y,
-                                       int width, int part, float eps, const TY* __restrict__ gate, int64_t ld_gate,
+                                       int64_t ldy, int width, int part, float eps, const TY* __restrict__ gate, int64_t ld_gate,
                                        int gate_act) {
     __shared__ float scratch[32];
     pdl_launch_dependents();
     pdl_wait();
     const int64_t base = (int64_t)blockIdx.x * width + (int64_t)blockIdx.y * part;
     const float* xr = x + base;
+    TY* yr = y + (int64_t)blockIdx.x * ldy + (int64_t)blockIdx.y * part;
     float ss = 0.0f;
     for (int c = threadIdx.x; c < part; c += blockDim.x) ss += xr[c] * xr[c];
     const float inv = 1.0f / sqrtf(block_sum(ss, scratch) / (float)part + eps);
@@ -191,18 +192,18 @@ __global__ void grouped_rmsnorm_kernel(const float* __restrict__ x, const float*
         const TY* gr = gate + (int64_t)blockIdx.x * ld_gate + (int64_t)blockIdx.y * part;
         for (int c = threadIdx.x; c < part; c += blockDim.x) {
             const float gv = to_f32(gr[c]);
-            y[base + c] = from_f32<TY>(xr[c] * inv * wr[c] * (gate_act == 1 ? gv : 1.0f) / (1.0f + expf(-gv)));
+            yr[c] = from_f32<TY>(xr[c] * inv * wr[c] * (gate_act == 1 ? gv : 1.0f) / (1.0f + expf(-gv)));
         }
         return;
     }
-    for (int c = threadIdx.x; c < part; c += blockDim.x) y[base + c] = from_f32<TY>(xr[c] * inv * wr[c]);
+    for (int c = threadIdx.x; c < part; c += blockDim.x) yr[c] = from_f32<TY>(xr[c] * inv * wr[c]);
 }
 
 // The same for parts of at most 1024 elements: one block a row, a warp a part (warps take parts in turn), so that a row of
 // many short parts (the heads of a recurrent layer) is one block instead of one tiny block a part.
 template <typename TY>
 __global__ void grouped_rmsnorm_warp_kernel(const float* __restrict__ x, const float* __restrict__ w, TY* __restrict__ y,
-                                            int width, int part, int groups, float eps, const TY* __restrict__ gate,
+                                            int64_t ldy, int width, int part, int groups, float eps, const TY* __restrict__ gate,
                                             int64_t ld_gate, int gate_act) {
     pdl_launch_dependents();
     pdl_wait();
@@ -232,7 +233,7 @@ __global__ void grouped_rmsnorm_warp_kernel(const float* __restrict__ x, const f
                     const float gv = to_f32(gr[c]);
                     o *= (gate_act == 1 ? gv : 1.0f) / (1.0f + expf(-gv));
                 }
-                y[base + c] = from_f32<TY>(o);
+                y[row * ldy + (int64_t)g * part + c] = from_f32<TY>(o);
             }
             if (32 * (k + 1) >= part) break;
         }
@@ -285,25 +286,27 @@ XS_API int xs_add_layernorm(float* h, const void* m, int m_dtype, const float* p
     return 0;
 }
 
-XS_API int xs_grouped_rmsnorm(const float* x, const float* w, void* y, int y_dtype, int rows, int width, int groups,
+// y's rows are `ldy` elements apart.
+XS_API int xs_grouped_rmsnorm(const float* x, const float* w, void* y, int64_t ldy, int y_dtype, int rows, int width, int groups,
                               float eps, const void* gate, int64_t ld_gate, int gate_act, cudaStream_t stream) {
     if (rows == 0) return 0;
     XS_REQUIRE(gate_act == 0 || gate_act == 1, "grouped_rmsnorm: gate activation %d (0 sigmoid, 1 silu)", gate_act);
     XS_REQUIRE(rows > 0 && width > 0 && groups > 0 && width % groups == 0, "grouped_rmsnorm: %d rows of %d in %d parts",
                rows, width, groups);
+    XS_REQUIRE(ldy >= width, "grouped_rmsnorm: rows of %d, %lld apart", width, (long long)ldy);
     XS_REQUIRE(groups <= 65535, "grouped_rmsnorm: %d parts exceed the grid limit", groups);
     const int part = width / groups;
     if (part <= 1024 && groups > 1) {
         const int warps = groups < 8 ? groups : 8;
         XS_DISPATCH_DTYPE(y_dtype, TY,
-                          xs_launch(grouped_rmsnorm_warp_kernel<TY>, dim3(rows), dim3(32 * warps), 0, stream, x, w, (TY*)y, width,
+                          xs_launch(grouped_rmsnorm_warp_kernel<TY>, dim3(rows), dim3(32 * warps), 0, stream, x, w, (TY*)y, ldy, width,
                                     part, groups, eps, (const TY*)gate, ld_gate, gate_act));
         XS_LAUNCH_CHECK("grouped_rmsnorm");
         return 0;
     }
     const int threads = part >= 1024 ? 256 : 128;
     XS_DISPATCH_DTYPE(y_dtype, TY,
-                      xs_launch(grouped_rmsnorm_kernel<TY>, dim3(rows, groups), dim3(threads), 0, stream, x, w, (TY*)y,
+                      xs_launch(grouped_rmsnorm_kernel<TY>, dim3(rows, groups), dim3(threads), 0, stream, x, w, (TY*)y, ldy,
                                 width, part, eps, (const TY*)gate, ld_gate, gate_act));
     XS_LAUNCH_CHECK("grouped_rmsnorm");
     return 0;

@@ -45,23 +45,23 @@ def _signatures(lib) -> None:
         "xs_zero_rows": [P, P, I, L, P],
         "xs_gemm_generic": [P, P, P, P, I, I, I, I, I, L, L, L, P],
         "xs_qk_norm_rope_store": [P, L, P, P, P, I, P, P, P, P, P, I, I, I, I, I, I, P, P, I, F, I, I, P],
-        "xs_attention_generic": [P, P, P, I, P, P, P, L, P, I, I, I, I, I, I, I, F, I, I, I, I, I, P],
+        "xs_attention_generic": [P, P, P, I, P, P, P, L, P, L, I, I, I, I, I, I, I, F, F, I, I, I, I, I, P],
         "xs_short_conv": [P, L, P, P, P, P, P, P, P, I, I, I, I, I, I, P],
         "xs_attention_mma": [P, P, P, I, P, P, P, L, P, P, L, I, I, I, I, I, I, I, F, I, I, P],
-        "xs_attention_tc": [P, P, L, P, I, P, P, P, L, P, I, I, I, I, I, I, I, I, F, I, I, I, I, I, P, P],
+        "xs_attention_tc": [P, P, L, P, I, P, P, P, L, P, L, I, I, I, I, I, I, I, I, F, F, I, I, I, I, I, P, P],
         "xs_gemm_small_m": [P, P, P, P, P, I, I, I, I, L, L, L, I, I, P, L, P],
         "xs_gemm_small_m_normed": [P, P, P, P, P, I, I, I, I, L, L, L, I, I, P, L, P, I, I, F, P, P, L, P, P],
         "xs_gemm_small_m_ex": [P, P, P, P, P, I, I, I, I, L, L, L, I, I, P, L, P, I, I, F, P, P, L, P,
                                P, P, P, P, P, P, I, I, P, P, P, P],
         "xs_gemm_small_m_rope": [P, P, P, P, I, I, I, L, L, L, P, I, I, F, P, P, P, I, P, P, P, P, P, I, I, I, I, F, P],
-        "xs_attention_mma_merged": [P, P, P, I, P, P, P, L, P, P, L, P, L, P, I, I, I, I, I, I, I, I, I, F, I, I, I, I, I, P],
+        "xs_attention_mma_merged": [P, P, P, I, P, P, P, L, P, L, P, L, P, L, P, I, I, I, I, I, I, I, I, I, F, F, I, I, I, I, I, P],
         "xs_gemm_tc": [P, P, P, P, I, I, I, I, I, L, L, L, I, P, L, P, P],
         "xs_argmax": [P, L, I, I, P, P, P],
         "xs_sample": [P, L, I, I, P, P, P, P, P, P, I, P, P],
         "xs_apply_penalties": [P, L, I, I, P, P, P, P, P, P, P],
         "xs_note_tokens": [P, P, I, I, P, P, I, P],
         "xs_add_layernorm": [P, P, I, P, P, P, I, P, I, I, F, F, P],
-        "xs_grouped_rmsnorm": [P, P, P, I, I, I, I, F, P, L, I, P],
+        "xs_grouped_rmsnorm": [P, P, P, L, I, I, I, I, F, P, L, I, P],
         "xs_clamped_glu": [P, P, I, I, I, L, F, F, F, I, P],
         "xs_gemm_tc_clamped": [P, P, P, I, I, I, I, L, L, L, F, F, F, P, P],
         "xs_gemm_tc_gelu": [P, P, P, I, I, I, I, L, L, L, P, P],
@@ -86,9 +86,13 @@ def _signatures(lib) -> None:
         "xs_depth_average": [P, L, P, I, P, L, P],
         "xs_rmsnorm_accumulate": [P, I, P, P, I, I, F, F, I, P],
         "xs_gated_delta_scan": [P, L, I, I, I, P, L, P, P, P, P, P, P, I, I, I, I, I, F, F, I, I, P],
-        "xs_moe_route_grouped": [P, I, I, I, I, P, I, I, I, F, I, F, I, I, P, P, P],
+        "xs_moe_route_grouped": [P, I, I, I, I, P, I, I, I, F, I, F, I, I, I, P, P, P],
         "xs_poly_norm": [P, L, P, P, I, I, F, I, P],
         "xs_stream_add": [P, P, P, I, I, P],
+        "xs_qkv_filter": [P, L, P, P, P, P, P, P, I, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, I, F, I, I, P],
+        "xs_token_mix": [P, L, P, P, P, P, P, P, I, I, I, I, P],
+        "xs_low_rank_decay": [P, L, P, I, P, P, I, I, I, I, I, F, P],
+        "xs_decay_scan": [P, L, P, L, P, L, P, P, P, P, P, P, P, L, P, P, L, I, I, I, I, F, F, I, P, P, I, P, P, P],
         "xs_mamba2_scan": [P, P, L, I, P, P, P, P, P, P, P, I, I, I, I, I, I, P],
         "xs_mamba2_scan_chunked": [P, P, L, I, P, P, P, P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, P],
     }
@@ -98,6 +102,8 @@ def _signatures(lib) -> None:
         fn.restype = c_int
     lib.xs_last_error.restype = ctypes.c_char_p
     lib.xs_last_error.argtypes = []
+    for name, args in (("xs_decay_scan_finishes", [c_int, c_int]), ("xs_decay_scan_blocks", [c_int, c_int, c_int])):
+        getattr(lib, name).restype, getattr(lib, name).argtypes = c_int, args
     lib.xs_uniform.restype = c_double
     lib.xs_uniform.argtypes = [c_uint64, c_uint64]
     lib.xs_abi_version.restype = c_int
@@ -400,6 +406,13 @@ def _need_pool(pool: torch.Tensor, kv_heads: int, page_size: int, head_dim: int,
         raise KernelError(f"cache is {tuple(pool.shape)}, expected [*, {', '.join(str(n) for n in shape)}]")
 
 
+def _need_heads(out: torch.Tensor, q: torch.Tensor) -> None:
+    """out [T, heads, DV] of q's type, a token's heads contiguous, any token stride."""
+    if (not out.is_cuda or out.dtype != q.dtype or out.dim() != 3 or out.shape[:2] != q.shape[:2] or out.stride(2) != 1
+            or out.stride(1) != out.shape[2]):
+        raise KernelError(f"attention: out is {tuple(out.shape)} {out.dtype} (strides {out.stride()}) for queries {tuple(q.shape)} {q.dtype}")
+
+
 def _need_gate(gate: Optional[torch.Tensor], q: torch.Tensor, heads: int, v_dim: int, channels: bool) -> int:
     """The gate's row stride (0 without one)."""
     if gate is None:
@@ -457,20 +470,21 @@ def qk_norm_rope_store(qkv: torch.Tensor, q_out: torch.Tensor, pool: Optional[to
 def attention_generic(q: torch.Tensor, pool: torch.Tensor, page_table: torch.Tensor, seq_of_token: torch.Tensor,
                       positions: torch.Tensor, gate: Optional[torch.Tensor], out: torch.Tensor, kv_heads: int,
                       page_size: int, scale: float, window: int, keep: int = 0, planes: int = 2, plus_one: bool = False,
-                      gate_channels: bool = False) -> None:
+                      gate_channels: bool = False, softcap: float = 0.0) -> None:
     """Attention over the paged cache, any even head size up to 256 (values: out's last dimension). `window` 0: every
     earlier key; W > 0: keys with pos - j < W or j < keep; -C: the query's own block of C positions. planes 1: the keys are
     the values. plus_one: the softmax's denominator has one more term of score 0. gate: logits per head, or with
-    gate_channels per channel."""
-    _need(q, "q"); _need(out, "out", q.dtype); _need(page_table, "page table", torch.int32)
+    gate_channels per channel. softcap > 0: scores are softcap * tanh(scale q.k / softcap). `out` may be columns of a wider
+    matrix (any token stride)."""
+    _need(q, "q"); _need_heads(out, q); _need(page_table, "page table", torch.int32)
     T, heads, D = q.shape
     DV = out.shape[2]
     _need_pool(pool, kv_heads, page_size, D, DV, planes, q.dtype)
     ld_gate = _need_gate(gate, q, heads, DV, gate_channels)
     _check(load().xs_attention_generic(
         q.data_ptr(), pool.data_ptr(), page_table.data_ptr(), page_table.shape[1], seq_of_token.data_ptr(),
-        positions.data_ptr(), _ptr(gate), ld_gate, out.data_ptr(), T, heads, kv_heads, D, DV, int(planes), page_size,
-        float(scale), int(window), int(keep), 1 if plus_one else 0, 1 if gate_channels else 0, _code(q), _stream()))
+        positions.data_ptr(), _ptr(gate), ld_gate, out.data_ptr(), out.stride(0), T, heads, kv_heads, D, DV, int(planes), page_size,
+        float(scale), float(softcap), int(window), int(keep), 1 if plus_one else 0, 1 if gate_channels else 0, _code(q), _stream()))
 
 
 def attention_mma_supports(head_dim: int, page_size: int, group: int, v_dim: int = 0) -> bool:
@@ -493,15 +507,15 @@ def attention_mma(q: torch.Tensor, pool: torch.Tensor, page_table: torch.Tensor,
                   scratch: Optional[torch.Tensor], n_seqs: int, max_q_len: int, kv_heads: int, page_size: int,
                   scale: float, window: int, splits: int, counters: Optional[torch.Tensor] = None,
                   bounded_waits: bool = False, keep: int = 0, planes: int = 2, plus_one: bool = False,
-                  gate_channels: bool = False) -> None:
+                  gate_channels: bool = False, softcap: float = 0.0) -> None:
     """Tensor-core attention over the paged bfloat16 cache. `scratch`: a byte buffer of at least
     attention_mma_scratch_bytes(tokens * heads, head_dim, splits) when splits > 1. `counters`: at least
     n_seqs * kv_heads zeroed int32 words that the kernel leaves zeroed; with them a decode step (one token a
     sequence) merges its key splits inside the attention kernel instead of in a second one. `bounded_waits`: a decode
     step at head size 64 may take the kernel that the TMA unit feeds; its waits are bounded, and one that gives up sets
     gemm_tc_status(device), which the caller then has to look at (tc_status_unread). The value size is out's last
-    dimension; `keep` to `gate_channels` as in attention_generic."""
-    _need(q, "q", torch.bfloat16); _need(out, "out", torch.bfloat16)
+    dimension; `keep` to `softcap` as in attention_generic."""
+    _need(q, "q", torch.bfloat16); _need_heads(out, q)
     _need(page_table, "page table", torch.int32)
     T, heads, D = q.shape
     DV = out.shape[2]
@@ -518,9 +532,9 @@ def attention_mma(q: torch.Tensor, pool: torch.Tensor, page_table: torch.Tensor,
         mark_bounded(q.device)
     _check(load().xs_attention_mma_merged(
         q.data_ptr(), pool.data_ptr(), page_table.data_ptr(), page_table.shape[1], cu_seqlens.data_ptr(),
-        kv_lens.data_ptr(), _ptr(gate), ld_gate, out.data_ptr(), _ptr(scratch), sbytes, _ptr(counters) if merged else None,
+        kv_lens.data_ptr(), _ptr(gate), ld_gate, out.data_ptr(), out.stride(0), _ptr(scratch), sbytes, _ptr(counters) if merged else None,
         pool.shape[0] if tma else 0, gemm_tc_status(q.device).data_ptr() if tma else None,
-        T, n_seqs, max_q_len, heads, kv_heads, D, DV, int(planes), page_size, float(scale), int(window), int(keep),
+        T, n_seqs, max_q_len, heads, kv_heads, D, DV, int(planes), page_size, float(scale), float(softcap), int(window), int(keep),
         1 if plus_one else 0, 1 if gate_channels else 0, int(splits), _stream()),
         kernels=2 if splits > 1 and not merged else 1)
 
@@ -532,19 +546,19 @@ def attention_tc_supports(head_dim: int, page_size: int, group: int) -> bool:
 def attention_tc(q: torch.Tensor, pool: torch.Tensor, page_table: torch.Tensor, cu_seqlens: torch.Tensor,
                  kv_lens: torch.Tensor, gate: Optional[torch.Tensor], out: torch.Tensor, n_seqs: int, max_q_len: int,
                  kv_heads: int, page_size: int, scale: float, window: int, max_kv_len: int = 0, keep: int = 0,
-                 planes: int = 2, plus_one: bool = False, gate_channels: bool = False) -> None:
+                 planes: int = 2, plus_one: bool = False, gate_channels: bool = False, softcap: float = 0.0) -> None:
     """Attention for prompts on the tcgen05 tensor cores (head size 64): the same operation as attention_mma with
     one key split. A wait that gives up inside the kernel sets gemm_tc_status(device). `max_kv_len` (the longest
     sequence's keys, 0 if unknown) only picks the order in which the kernel's CTAs start."""
-    _need(q, "q", torch.bfloat16); _need(out, "out", torch.bfloat16); _need(page_table, "page table", torch.int32)
+    _need(q, "q", torch.bfloat16); _need_heads(out, q); _need(page_table, "page table", torch.int32)
     T, heads, D = q.shape
     _need_pool(pool, kv_heads, page_size, D, out.shape[2], planes, torch.bfloat16)
     ld_gate = _need_gate(gate, q, heads, D, gate_channels)
     mark_bounded(q.device)
     _check(load().xs_attention_tc(
         q.data_ptr(), pool.data_ptr(), pool.shape[0], page_table.data_ptr(), page_table.shape[1], cu_seqlens.data_ptr(),
-        kv_lens.data_ptr(), _ptr(gate), ld_gate, out.data_ptr(), T, n_seqs, max_q_len, heads, kv_heads, D, int(planes), page_size,
-        float(scale), int(window), int(keep), 1 if plus_one else 0, 1 if gate_channels else 0, int(max_kv_len), gemm_tc_status(q.device).data_ptr(), _stream()))
+        kv_lens.data_ptr(), _ptr(gate), ld_gate, out.data_ptr(), out.stride(0), T, n_seqs, max_q_len, heads, kv_heads, D, int(planes), page_size,
+        float(scale), float(softcap), int(window), int(keep), 1 if plus_one else 0, 1 if gate_channels else 0, int(max_kv_len), gemm_tc_status(q.device).data_ptr(), _stream()))
 
 
 def gemm_small_m_supports(M: int, K: int, ldx: int, ldw: int) -> bool:
@@ -875,12 +889,12 @@ def grouped_rmsnorm(x: torch.Tensor, w: torch.Tensor, y: torch.Tensor, groups: i
     or by silu(gate) with gate_act "silu"."""
     if gate_act not in ("sigmoid", "silu"):
         raise KernelError(f"grouped_rmsnorm: gate activation '{gate_act}' (sigmoid, silu)")
-    _need(x, "x", torch.float32); _need(w, "w", torch.float32); _need(y, "y")
-    if y.shape != x.shape or w.numel() != x.shape[1]:
+    _need(x, "x", torch.float32); _need(w, "w", torch.float32)
+    if y.shape != x.shape or w.numel() != x.shape[1] or not y.is_cuda or y.stride(1) != 1:
         raise KernelError(f"grouped_rmsnorm: x {tuple(x.shape)}, w {tuple(w.shape)}, y {tuple(y.shape)}")
     if gate is not None and (gate.dtype != y.dtype or gate.stride(1) != 1 or gate.shape[0] != x.shape[0] or gate.shape[1] < x.shape[1]):
         raise KernelError(f"grouped_rmsnorm: gate {tuple(gate.shape)} {gate.dtype} for y {tuple(y.shape)} {y.dtype}")
-    _check(load().xs_grouped_rmsnorm(x.data_ptr(), w.data_ptr(), y.data_ptr(), _code(y), x.shape[0], x.shape[1],
+    _check(load().xs_grouped_rmsnorm(x.data_ptr(), w.data_ptr(), y.data_ptr(), y.stride(0), _code(y), x.shape[0], x.shape[1],
                                      int(groups), float(eps), _ptr(gate), 0 if gate is None else gate.stride(0),
                                      1 if gate_act == "silu" else 0, _stream()))
 
@@ -960,13 +974,13 @@ def moe_route(logits: torch.Tensor, top: int, ids: torch.Tensor, wts: torch.Tens
 def moe_route_grouped(logits: torch.Tensor, top: int, ids: torch.Tensor, wts: torch.Tensor, experts: Optional[int] = None,
                       correction: Optional[torch.Tensor] = None, groups: int = 1, keep: int = 1, group_top: int = 2,
                       scale: float = 1.0, renorm: bool = False, score: str = "sigmoid", real: Optional[int] = None,
-                      renorm_eps: float = 0.0) -> None:
+                      renorm_eps: float = 0.0, squared: bool = False) -> None:
     """Per row of float32 logits: scores s = sigmoid(logit), choice scores c = s + correction; the experts stand in
     `groups` equal groups of neighbours, of which the `keep` with the largest sum of their `group_top` largest choice
     scores stay open; the `top` open experts with the largest c (ties: the lower index) go into ids, their s (times
     `scale`; divided by their sum + `renorm_eps` with `renorm`) into wts. `score` "softmax": s is the softmax over all `experts` logits
     instead. `real`: only the first so many experts have weights; a choice of a later one is written as id -1 (its input
-    passes, times its weight)."""
+    passes, times its weight). `squared`: the weights' squares go into wts."""
     _need(logits, "router logits", torch.float32); _need(ids, "ids", torch.int32); _need(wts, "weights", torch.float32)
     if score not in ("sigmoid", "softmax"):
         raise KernelError(f"moe_route_grouped: score '{score}' (sigmoid, softmax)")
@@ -979,7 +993,7 @@ def moe_route_grouped(logits: torch.Tensor, top: int, ids: torch.Tensor, wts: to
     if ids.numel() < T * top or wts.numel() < T * top:
         raise KernelError(f"moe_route_grouped: {T} tokens x top {top} do not fit ids {ids.numel()} / weights {wts.numel()}")
     _check(load().xs_moe_route_grouped(logits.data_ptr(), ld, T, E, int(top), _ptr(correction), int(groups), int(keep),
-                                       int(group_top), float(scale), 1 if renorm else 0, float(renorm_eps), 1 if score == "softmax" else 0,
+                                       int(group_top), float(scale), 1 if renorm else 0, float(renorm_eps), 1 if squared else 0, 1 if score == "softmax" else 0,
                                        E if real is None else int(real), ids.data_ptr(), wts.data_ptr(), _stream()))
 
 
@@ -1498,3 +1512,138 @@ def gated_delta_scan(qkv: torch.Tensor, q_col: int, k_col: int, v_col: int, ab: 
                                       ab.stride(0), a_log.data_ptr(), dt_bias.data_ptr(), state.data_ptr(),
                                       cu_seqlens.data_ptr(), slots.data_ptr(), y.data_ptr(), slots.numel(), int(heads),
                                       int(key_heads), int(dim), int(vdim), float(q_scale), float(unit_eps), int(T), _code(qkv), _stream()))
+
+
+# ------------------------------------------------ filtered projections, neighbouring tokens, memories with a decay per row
+def qkv_filter(proj: torch.Tensor, bias: Optional[torch.Tensor], taps: torch.Tensor, state: Optional[torch.Tensor], q_out: torch.Tensor,
+               pool: torch.Tensor, page_table: torch.Tensor, seq_of_token: torch.Tensor, positions: torch.Tensor, cu_seqlens: torch.Tensor,
+               slots: torch.Tensor, q_w: Optional[torch.Tensor], k_w: Optional[torch.Tensor], rope: Optional[torch.Tensor], heads: int,
+               kv_heads: int, head_dim: int, v_dim: int, page_size: int, eps: float, q_count: int, k_count: int,
+               all_single: bool = False) -> None:
+    """Columns [q heads | k heads | v heads] of proj, plus `bias`, through a causal filter per channel (taps [n, channels]: row b
+    looks b tokens back; zeros before a sequence's first token; earlier rows from `state` [*, n - 1, channels], which then moves
+    on), then queries and keys normed over all heads together (weights q_w [heads * head_dim], k_w; the means are over q_count
+    and k_count channels) and rotated: queries to q_out, keys and filtered values into the cache's pages (csrc/qkv_filter.cu).
+    `all_single`: every sequence brings exactly one token."""
+    T = proj.shape[0]
+    C = heads * head_dim + kv_heads * (head_dim + v_dim)
+    n = taps.shape[0]
+    _need(q_out, "q_out", proj.dtype); _need(taps, "taps", torch.float32); _need(page_table, "page table", torch.int32)
+    if not proj.is_cuda or proj.stride(1) != 1 or proj.shape[1] < C or tuple(q_out.shape) != (T, heads, head_dim) or taps.shape[1] != C:
+        raise KernelError(f"qkv_filter: rows {tuple(proj.shape)}, q_out {tuple(q_out.shape)}, taps {tuple(taps.shape)} for {C} channels")
+    _need_pool(pool, kv_heads, page_size, head_dim, v_dim, 2, proj.dtype)
+    if n > 1:
+        _need(state, "filter state", proj.dtype)
+        if tuple(state.shape[1:]) != (n - 1, C):
+            raise KernelError(f"qkv_filter: state is {tuple(state.shape)}, expected [*, {n - 1}, {C}]")
+    for v, name, size in ((q_w, "q norm", heads * head_dim), (k_w, "k norm", kv_heads * head_dim), (bias, "bias", C)):
+        if v is not None:
+            _need(v, name, torch.float32)
+            if v.numel() < size:
+                raise KernelError(f"qkv_filter: {name} has {v.numel()} entries, {size} are needed")
+    if rope is not None:
+        _need(rope, "rope table", torch.float32)
+        if tuple(rope.shape[1:]) != (head_dim // 2, 2):
+            raise KernelError(f"rope table is {tuple(rope.shape)}, expected [*, {head_dim // 2}, 2]")
+    _check(load().xs_qkv_filter(proj.data_ptr(), proj.stride(0), _ptr(bias), taps.data_ptr(), _ptr(state) if n > 1 else None,
+                                q_out.data_ptr(), pool.data_ptr(), page_table.data_ptr(), page_table.shape[1], seq_of_token.data_ptr(),
+                                positions.data_ptr(), cu_seqlens.data_ptr(), slots.data_ptr(), _ptr(q_w), _ptr(k_w), _ptr(rope), T,
+                                slots.numel(), heads, kv_heads, head_dim, v_dim, n, int(q_count), int(k_count), page_size, float(eps),
+                                1 if all_single else 0, _code(proj), _stream()),
+           kernels=2 if n > 1 and not all_single else 1)
+
+
+def token_mix(x: torch.Tensor, state: torch.Tensor, mu: torch.Tensor, out: torch.Tensor, seq_of_token: torch.Tensor,
+              cu_seqlens: torch.Tensor, slots: torch.Tensor) -> None:
+    """out[s, t] = x[t] + (the token before t in its sequence - x[t]) * mu[s]; before a step's first token stands `state`
+    [*, width] (x's type; zeros at a sequence's start), which then takes the sequence's last row."""
+    _need(state, "previous tokens", x.dtype); _need(mu, "mixes", torch.float32); _need(out, "out", x.dtype)
+    T, W = x.shape
+    n = mu.shape[0]
+    if not x.is_cuda or x.stride(1) != 1 or mu.shape[1] != W or tuple(out.shape) != (n, T, W) or tuple(state.shape[1:]) != (W,):
+        raise KernelError(f"token_mix: x {tuple(x.shape)}, mixes {tuple(mu.shape)}, out {tuple(out.shape)}, state {tuple(state.shape)}")
+    _check(load().xs_token_mix(x.data_ptr(), x.stride(0), state.data_ptr(), mu.data_ptr(), out.data_ptr(), seq_of_token.data_ptr(),
+                               cu_seqlens.data_ptr(), slots.data_ptr(), T, W, n, _code(x), _stream()))
+
+
+DECAY_KINDS = {"double_exp": 0, "rooted_sigmoid": 1}
+
+
+def low_rank_decay(z: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor], out: torch.Tensor, kind: str, hidden_tanh: bool = False,
+                   power: float = 1.0) -> None:
+    """out[t, c] = exp(-exp(v)) ("double_exp") or sigmoid(v)^power ("rooted_sigmoid") with v = w[c] . f(z[t]) + bias[c], f nothing
+    or tanh. z [T, rank] and out [T, channels] float32, w [channels, rank] in the activation type; everything float32."""
+    if kind not in DECAY_KINDS:
+        raise KernelError(f"low_rank_decay: kind '{kind}' ({', '.join(DECAY_KINDS)})")
+    _need(w, "decay weight"); _need(out, "out", torch.float32)
+    C, R = w.shape
+    T = out.shape[0]
+    if not z.is_cuda or z.dtype != torch.float32 or z.stride(1) != 1 or z.shape[0] != T or z.shape[1] < R or out.shape[1] != C:
+        raise KernelError(f"low_rank_decay: z {tuple(z.shape)} {z.dtype}, w {tuple(w.shape)}, out {tuple(out.shape)}")
+    if bias is not None:
+        _need(bias, "bias", torch.float32)
+        if bias.numel() != C:
+            raise KernelError(f"low_rank_decay: a bias of {bias.numel()} for {C} channels")
+    _check(load().xs_low_rank_decay(z.data_ptr(), z.stride(0), w.data_ptr(), _code(w), _ptr(bias), out.data_ptr(), T, C, R,
+                                    1 if hidden_tanh else 0, DECAY_KINDS[kind], float(power), _stream()))
+
+
+def decay_scan_finishes(dim: int, vdim: int) -> bool:
+    """Whether decay_scan can norm and gate the heads' outputs itself."""
+    return bool(load().xs_decay_scan_finishes(dim, vdim))
+
+
+def decay_scan_blocks(heads: int, dim: int, vdim: int) -> int:
+    """CTAs of one sequence or chunk."""
+    return int(load().xs_decay_scan_blocks(heads, dim, vdim))
+
+
+def decay_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, decay: torch.Tensor, state: torch.Tensor, cu_seqlens: torch.Tensor,
+               slots: torch.Tensor, heads: int, dim: int, vdim: int, q_scale: float = 1.0, bonus: Optional[torch.Tensor] = None,
+               y: Optional[torch.Tensor] = None, out: Optional[torch.Tensor] = None, norm_w: Optional[torch.Tensor] = None,
+               gate: Optional[torch.Tensor] = None, eps: float = 0.0, chunks=None) -> None:
+    """S <- diag(decay[t]) S + k v^T per head over a step's tokens, sequence by sequence from each slot's state [*, heads, dim, vdim]
+    (float32): o = S^T (q_scale q) behind the write, or with `bonus` [heads, dim] before it with bonus times the token's own pair
+    added (csrc/decay_scan.cu). q, k, v: matrices whose first heads * dim (v: heads * vdim) columns are used; decay
+    [T, heads * dim] float32. The float32 outputs go to y [T, heads * vdim]; or (decay_scan_finishes) `out` takes them divided by
+    their head's root mean square (eps), times norm_w [heads * vdim], times silu(gate). `chunks` (list [n, 3] int32, first chunk of
+    each sequence, scratch [n, heads, dim, vdim] and [n, heads, dim] float32): the chunks run side by side."""
+    _need(decay, "decay", torch.float32); _need(state, "state", torch.float32)
+    T = q.shape[0]
+    for t, name, cols in ((q, "q", heads * dim), (k, "k", heads * dim), (v, "v", heads * vdim)):
+        if not t.is_cuda or t.dim() != 2 or t.stride(1) != 1 or t.shape[0] != T or t.shape[1] < cols or t.dtype != q.dtype:
+            raise KernelError(f"decay_scan: {name} is {tuple(t.shape)} {t.dtype} for {T} tokens of {cols} columns")
+    if tuple(decay.shape) != (T, heads * dim) or tuple(state.shape[1:]) != (heads, dim, vdim):
+        raise KernelError(f"decay_scan: decay {tuple(decay.shape)}, state {tuple(state.shape)} for {heads} heads of {dim} x {vdim}")
+    if bonus is not None:
+        _need(bonus, "bonus", torch.float32)
+        if bonus.numel() != heads * dim:
+            raise KernelError(f"decay_scan: a bonus of {bonus.numel()} entries for {heads} heads of {dim}")
+    if y is not None:
+        _need(y, "y", torch.float32)
+        if tuple(y.shape) != (T, heads * vdim):
+            raise KernelError(f"decay_scan: y {tuple(y.shape)} for {T} tokens of {heads * vdim}")
+    else:
+        _need(norm_w, "norm weight", torch.float32)
+        for t, name in ((out, "out"), (gate, "gate")):
+            if t is None or t.dtype != q.dtype or t.stride(1) != 1 or t.shape[0] != T or t.shape[1] < heads * vdim:
+                raise KernelError(f"decay_scan: {name} must hold {T} rows of {heads * vdim} in the activation type")
+        if norm_w.numel() != heads * vdim:
+            raise KernelError(f"decay_scan: a norm weight of {norm_w.numel()} for rows of {heads * vdim}")
+    chunk_args = (None, None, 0, None, None)
+    if chunks is not None:
+        chunk_seq, first_chunk, chunk_state, chunk_decay = chunks
+        n = chunk_seq.shape[0]
+        _need(chunk_seq, "chunk list", torch.int32); _need(first_chunk, "first chunks", torch.int32)
+        _need(chunk_state, "chunk states", torch.float32); _need(chunk_decay, "chunk decays", torch.float32)
+        if (tuple(chunk_state.shape) != (n, heads, dim, vdim) or tuple(chunk_decay.shape) != (n, heads, dim)
+                or first_chunk.numel() != cu_seqlens.numel()):
+            raise KernelError(f"decay_scan: chunk scratch {tuple(chunk_state.shape)} for {n} chunks")
+        chunk_args = (chunk_seq.data_ptr(), first_chunk.data_ptr(), n, chunk_state.data_ptr(), chunk_decay.data_ptr())
+    finish = y is None
+    _check(load().xs_decay_scan(q.data_ptr(), q.stride(0), k.data_ptr(), k.stride(0), v.data_ptr(), v.stride(0), decay.data_ptr(),
+                                _ptr(bonus), state.data_ptr(), cu_seqlens.data_ptr(), slots.data_ptr(), _ptr(y),
+                                _ptr(out) if finish else None, out.stride(0) if finish else 0, _ptr(norm_w) if finish else None,
+                                _ptr(gate) if finish else None, gate.stride(0) if finish else 0, cu_seqlens.numel() - 1, heads, dim,
+                                vdim, float(q_scale), float(eps), _code(q), *chunk_args, _stream()),
+           kernels=3 if chunks is not None else 1)

@@ -13,7 +13,8 @@ from .poly_norm import PolyNormUnit
 from .mlstm import MLstmMixer
 from .lightning import LightningMixer
 from .gated_delta import GatedDeltaMixer
-from .parallel import ParallelMixer
+from .decay_memory import GatedLinearMixer, TimeMixingMixer
+from .parallel import ParallelMixer, SummedMixer
 from .embedding import LearnedPositionEmbedding, PairHashEmbedding
 from .block import Block, BranchNormBlock, GatedPreNormBlock, ResidualStream
 
@@ -21,4 +22,5 @@ __all__ = ["FeedForward", "KVNeed", "Mixer", "Norm", "RMSNorm", "Part", "StateNe
            "AttentionMixer", "ShortConvMixer", "SwiGLU", "Block", "ResidualStream", "LayerNorm", "ScaledRotaryTable",
            "LatentAttentionMixer", "Mamba2Mixer", "ClampedGLU", "RoutedExperts", "SquaredRelu", "MLstmMixer",
            "PairHashEmbedding", "BranchNormBlock", "GatedDeltaMixer", "ParallelMixer", "LearnedPositionEmbedding",
-           "GatedPreNormBlock", "LightningMixer", "PolyNormUnit"]
+           "GatedPreNormBlock", "LightningMixer", "PolyNormUnit", "GatedLinearMixer",
+           "TimeMixingMixer", "SummedMixer"]

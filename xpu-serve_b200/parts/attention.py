@@ -24,7 +24,10 @@ norms, with a weight of ones); keys that are the values (`shared_kv`: one vector
 loaded once for both products); one added to the softmax's denominator (`plus_one`); a gate on every
 output channel (`out_gate`, in the attention kernels' epilogues); a factor per head on the scores
 (`head_temp`, on the queries as they are stored). A rotation of some of a head's channels, or of
-neighbouring ones, is brought into the kernels' pairing by the order of the weights' rows (`channel_layout`).
+neighbouring ones, is brought into the kernels' pairing by the order of the weights' rows (`channel_layout`). Causal filters
+over time on q, k and v (`qkv_taps`; their last inputs are part of a sequence's state) and norms over whole projections
+(`qk_norm_all`) run with the rotation and the cache write in one kernel (csrc/qkv_filter.cu); a soft cap on the scores
+(`softcap`) in the attention kernels; an output bias (`o_bias`) in the output product.
 """
 from __future__ import annotations
 
@@ -36,7 +39,7 @@ import torch
 from .. import registry
 from ..config.spec import RopeSpec, ScaledRopeSpec
 from ..ops import lib as ops
-from .base import KVNeed, Mixer, TensorSpec
+from .base import KVNeed, Mixer, StateNeed, TensorSpec
 
 
 def decode_splits(tiles: int, blocks: int, slots: int, fixed: float = 2.0) -> int:
@@ -122,6 +125,7 @@ class AttentionMixer(Mixer):
     kind = "attention"
     fuses_norm = True
     fixed_shape_ok = True
+    concat_output = True
 
     @classmethod
     def tensors(cls, spec) -> Dict[str, TensorSpec]:
@@ -149,6 +153,14 @@ class AttentionMixer(Mixer):
                 out[n["k_bias"]] = TensorSpec((kd,), role="vector")
             if own_v:
                 out[n["v_bias"]] = TensorSpec((spec.kv_heads * vd,), role="vector")
+        if spec.qkv_taps:
+            for key, rows in (("q_conv", qd), ("k_conv", kd), ("v_conv", spec.kv_heads * vd)):
+                out[n[key]] = TensorSpec((rows, spec.qkv_taps), init="uniform:-0.5:0.5", role="vector")
+        if spec.qk_norm_all:
+            out[n["q_norm"]] = TensorSpec((qd,), init="ones", role="vector")
+            out[n["k_norm"]] = TensorSpec((kd,), init="ones", role="vector")
+        if spec.o_bias:
+            out[n["o_bias"]] = TensorSpec((spec.hidden,), role="vector")
         if spec.head_temp:
             out[n["temp"]] = TensorSpec((spec.heads,), init="uniform:0.5:1.5", role="vector")
         return out
@@ -158,8 +170,11 @@ class AttentionMixer(Mixer):
         # (a block mask keeps every key: a reader of this cache may have another mask)
         D, DV = head_sizes(spec)
         window = spec.window if not spec.chunk else 0
-        return KVNeed(spec.kv_heads, D, window, planes=1 if spec.shared_kv else 2, keep_first=spec.keep_first if window > 0 else 0,
-                      v_dim=DV if DV != D else 0)
+        kv = KVNeed(spec.kv_heads, D, window, planes=1 if spec.shared_kv else 2, keep_first=spec.keep_first if window > 0 else 0,
+                    v_dim=DV if DV != D else 0)
+        if spec.qkv_taps > 1:
+            return kv, StateNeed((spec.qkv_taps - 1, spec.heads * D + spec.kv_heads * (D + DV)), "compute")
+        return kv
 
     def __init__(self, spec, weights: Dict[str, torch.Tensor], rt):
         vd = spec.v_dim or spec.head_dim
@@ -180,6 +195,12 @@ class AttentionMixer(Mixer):
             raise ValueError("attention: a layer has learned or unit q/k norms, a gate per head or per channel, not both")
         if spec.unit_qk and getattr(getattr(spec.position, "scaling", None), "mscale_k", 0.0) != 0.0:
             raise ValueError("attention: unit queries and keys behind a rotation that changes lengths are not supported")
+        self.filtered = spec.qkv_taps > 0 or spec.qk_norm_all      # q, k and v pass the kernel of csrc/qkv_filter.cu
+        if self.filtered and (not spec.own_kv or spec.shared_kv or spec.qk_norm or spec.unit_qk or spec.head_temp):
+            raise ValueError("attention: filters and norms over whole projections need keys and values of the layer's own, no other norm "
+                             "and no factor on the scores")
+        if not 0 <= spec.qkv_taps <= 16 or not spec.softcap >= 0.0:
+            raise ValueError(f"attention: {spec.qkv_taps} taps (at most 16), soft cap {spec.softcap}")
         if not spec.scale > 0.0 or spec.keep_first < 0:
             raise ValueError("attention: the scale must be positive and keep_first not negative")
         self.spec, self.rt = spec, rt
@@ -190,7 +211,7 @@ class AttentionMixer(Mixer):
         self.kv_cols = spec.kv_heads * (D + (DV if self.planes == 2 else 0))
         # what the kernels need beside the window: passed on to each of them
         self.options = dict(keep=int(spec.keep_first) if spec.window > 0 else 0, planes=self.planes, plus_one=bool(spec.plus_one),
-                            gate_channels=bool(spec.out_gate))
+                            gate_channels=bool(spec.out_gate), softcap=float(spec.softcap))
         # the per-head norm over head_dim channels, computed over D: sum / D + eps' = (head_dim / D) (sum / head_dim + eps)
         self.qk_eps = float(spec.qk_norm_eps) * spec.head_dim / D
         norm_scale = (spec.head_dim / D) ** 0.5
@@ -242,6 +263,17 @@ class AttentionMixer(Mixer):
         if DV != vd:        # zero columns where the padded value channels stand
             w_o = values(w_o.t().contiguous(), spec.heads).t().contiguous()
         self.w_o = rt.matrix(w_o)
+        self.b_o = rt.vector(weights[n["o_bias"]]) if spec.o_bias else None
+
+        self.taps = None
+        if self.filtered:
+            # [taps, channels], row b for the tap that looks b tokens back (one tap of 1 where only the norms are wanted)
+            def filters(key, arrange, heads, d):
+                if not spec.qkv_taps:
+                    return arrange(torch.ones(heads * d, 1), heads)
+                return arrange(weights[n[key]].to(torch.float32).reshape(heads * d, spec.qkv_taps), heads)
+            self.taps = rt.vector(torch.cat([filters("q_conv", keys, spec.heads, hd), filters("k_conv", keys, spec.kv_heads, hd),
+                                             filters("v_conv", values, spec.kv_heads, vd)], 0).flip(1).t())
 
         def norm_weight(w: torch.Tensor):
             return rt.vector(keys(w.to(torch.float32), 1) * norm_scale)
@@ -250,6 +282,9 @@ class AttentionMixer(Mixer):
         if spec.qk_norm:
             self.q_norm = norm_weight(weights[n["q_norm"]])
             self.k_norm = norm_weight(weights[n["k_norm"]]) if spec.own_kv else None
+        elif spec.qk_norm_all:
+            self.q_norm = rt.vector(keys(weights[n["q_norm"]].to(torch.float32), spec.heads))
+            self.k_norm = rt.vector(keys(weights[n["k_norm"]].to(torch.float32), spec.kv_heads))
         elif spec.unit_qk:
             self.q_norm = self.k_norm = norm_weight(torch.ones(hd))
         self.q_scale = rt.vector(weights[n["temp"]]) if spec.head_temp else None
@@ -261,7 +296,23 @@ class AttentionMixer(Mixer):
     def takes_prenormed(self, rows: int) -> bool:
         return (self.w_qkvg is not None and self.rt.few_rows_shape(rows, self.w_qkvg) and self.w_qkvg.shape[1] % 8 == 0)
 
+    def scale_output(self, s: float) -> bool:
+        """What the heads leave is linear in the values, and those in their filters, which are float32."""
+        if self.taps is None:
+            return s == 1.0
+        self.taps[:, self.q_dim + self.spec.kv_heads * self.D:] *= s
+        return True
+
     def forward(self, x, step, cache, into=None) -> torch.Tensor:
+        T = x.shape[0]
+        o = self.rt.ws.get("attn_o", (T, self.o_dim), self.rt.act_dtype)
+        self.heads(x, step, cache, o)
+        if into is not None:
+            return into.product(o, self.w_o, self.b_o)
+        return self.rt.linear(o, self.w_o, "mixer_out", self.b_o)
+
+    def heads(self, x, step, cache, out) -> None:
+        """Everything in front of the output projection, into `out` [tokens, o_dim] (columns of any matrix)."""
         s, rt = self.spec, self.rt
         T = x.shape[0]
         if cache is None or cache.storage is None:
@@ -280,7 +331,16 @@ class AttentionMixer(Mixer):
         table = step.page_tables[cache.group]
         rope = self.position.table(step.max_positions) if self.position is not None else None
         q = rt.ws.get("attn_q", (T, s.heads, D), rt.act_dtype)
-        if step.decode and D == DV and self.planes == 2 and self.q_scale is None and rt.rope_behind_product(x, w_in, D):
+        if self.filtered:
+            if not cache.owner or len(cache) != (2 if s.qkv_taps > 1 else 1):
+                raise RuntimeError("attention with filtered projections keeps its own keys, values and filter inputs")
+            # (the filter's kernel adds the biases: a filter starts from zeros, not from biases)
+            proj = rt.linear(x, w_in, "attn_qkv")
+            ops.qkv_filter(proj, b_in, self.taps, cache[1].storage if s.qkv_taps > 1 else None, q, cache[0].storage, table,
+                           step.seq_of_token, step.positions, step.cu_seqlens, step.slots, self.q_norm, self.k_norm, rope, s.heads,
+                           s.kv_heads, D, DV, step.page_size, s.qk_norm_eps, s.heads * s.head_dim, s.kv_heads * s.head_dim,
+                           all_single=step.decode)
+        elif step.decode and D == DV and self.planes == 2 and self.q_scale is None and rt.rope_behind_product(x, w_in, D):
             # one token a sequence: the per-head norms, the rotation and the cache write run behind the product, in its kernel
             proj = rt.ws.get("attn_qkv", (T, w_in.shape[0]), rt.act_dtype)
             rt.few_rows_rope(x, w_in, proj, b_in, q_out=q, pool=cache.storage if cache.owner else None,
@@ -294,12 +354,8 @@ class AttentionMixer(Mixer):
             ops.qk_norm_rope_store(proj, q, cache.storage, table, step.seq_of_token, step.positions, self.q_norm,
                                    self.k_norm, rope, s.heads, s.kv_heads, D, step.page_size, self.qk_eps,
                                    write_kv=cache.owner, v_dim=DV, planes=self.planes, q_scale=self.q_scale, bias=late)
-        o = rt.ws.get("attn_o", (T, s.heads, DV), rt.act_dtype)
         gate = proj[:, gate_at:] if s.head_gate or s.out_gate else None
-        self.attend(q, cache, table, step, gate, o)
-        if into is not None:
-            return into.product(o.view(T, self.o_dim), self.w_o)
-        return rt.linear(o.view(T, self.o_dim), self.w_o, "mixer_out")
+        self.attend(q, cache, table, step, gate, out.unflatten(1, (s.heads, DV)))
 
     def attend(self, q, cache, table, step, gate, o) -> None:
         s, rt, D, DV, mask = self.spec, self.rt, self.D, self.DV, self.mask

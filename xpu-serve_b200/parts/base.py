@@ -31,6 +31,10 @@ a parts.block.Prenormed (the stream times the norm's weight, with the row scale 
 which it may hand to `rt.linear` / `rt.few_rows_product` only; and when `into` is given it sends its
 last product through `into.product(act, w, bias)` (which adds it to the stream inside the product's
 kernel) and returns None. Parts without the flag get the normed tensor and return their branch.
+A mixer whose class sets `concat_output = True` can leave its output projection to a mixer around it
+(parts/parallel.py): `heads(x, step, cache, out)` writes what the projection would read into `out` [tokens, o_dim]
+(rows of a wider matrix); `w_o` [hidden, o_dim] and `b_o` (None or float32 [hidden]) are the projection, and
+`scale_output(s)` multiplies what `heads` writes by a constant, or says False if it cannot.
 Such a part also says, per number of rows, whether the product that reads its input runs on the few-row kernel
 (`takes_prenormed(rows)`): only then is it handed a Prenormed; otherwise it gets the normed tensor, and still `into`.
 `step` is engine.step.StepContext (which tokens belong to which sequence, where each
@@ -47,6 +51,8 @@ class TensorSpec:
     shape: Tuple[int, ...]
     init: str = "normal"     # random-weights mode: "normal" N(0, std) | "ones" | "zeros" | "uniform:lo:hi"
     role: str = "matrix"     # "matrix": held in the compute dtype; "vector": held in float32
+    free: Tuple[Tuple[int, str], ...] = ()   # (axis, label): sizes that the checkpoint decides; tensors of a layer with the same
+                             # label agree about it, and `shape` names what a model with random weights gets
 
 
 @dataclass(frozen=True)
@@ -72,6 +78,7 @@ class StateNeed:
 class Part:
     kind: str = ""
     fuses_norm: bool = False    # see the module text: takes a Prenormed input and an `into` sink
+    concat_output: bool = False  # (mixers) see the module text: heads, w_o, b_o, o_dim, scale_output
     # Whether the part's code for prompt steps can be captured in a CUDA graph that serves any lengths up to the step's
     # bounds (`step.fixed_shape`): no host-side loop over `step.q_lens_host`, no host sync, sizes from the tensors'
     # shapes and `step.max_q_len` only. The library's parts say yes; the model captures single-sequence prompt steps

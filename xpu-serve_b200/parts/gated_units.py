@@ -15,6 +15,8 @@ RoutedExperts:  `experts` gated feed-forwards without biases (SwiGLU, or clamped
                 `score` "softmax_all": scores softmax over all router outputs, chosen by score plus a correction, weighted
                 by the scores as they are or over their sum; with `identity` the router's last outputs stand for the token's input itself
                 (such a choice takes no place in the plan; the combine kernel adds weight times input).
+                `weight_on` "input": an expert is fed its weight times the token. A squared-ReLU expert is homogeneous of
+                degree two, expert(w x) = w^2 expert(x) for w >= 0, so the routing kernel hands out the squared weights.
 """
 from __future__ import annotations
 
@@ -80,7 +82,8 @@ class SquaredRelu(FeedForward):
         self.w_up = rt.matrix(weights[spec.names["up"]])
         self.w_down = rt.matrix(weights[spec.names["down"]])
 
-    def forward(self, y, step) -> torch.Tensor:
+    def forward(self, y, step, name: str = "ffn_out") -> torch.Tensor:
+        """`name`: the scratch buffer that takes the result (a unit inside another feed-forward names its own)."""
         rt = self.rt
         act = rt.ws.get("ffn_act", (y.shape[0], self.spec.intermediate), rt.act_dtype)
         if rt.few_rows(y, self.w_up):
@@ -92,7 +95,7 @@ class SquaredRelu(FeedForward):
         else:
             up = rt.linear(y, self.w_up, "ffn_up")
             ops.relu_squared(up, act)
-        return rt.linear(act, self.w_down, "ffn_out")
+        return rt.linear(act, self.w_down, name)
 
 
 class RoutedExperts(FeedForward):
@@ -129,6 +132,9 @@ class RoutedExperts(FeedForward):
             raise ValueError("routed experts: identity outputs belong to softmax_all scores")
         if spec.score == "softmax" and (spec.correction or spec.groups != 1):
             raise ValueError("routed experts: a correction and groups belong to sigmoid scores or to the softmax over all outputs")
+        if spec.weight_on not in ("output", "input") or (spec.weight_on == "input" and (spec.activation != "relu_squared" or spec.score == "softmax"
+                                                                                       or self.identity)):
+            raise ValueError("routed experts: weights on the experts' inputs need squared-ReLU experts and scores over all outputs")
         outputs = spec.experts + self.identity
         if spec.groups < 1 or outputs % spec.groups != 0 or not 1 <= spec.keep_groups <= spec.groups \
                 or spec.keep_groups * (outputs // spec.groups) < spec.top:
@@ -182,11 +188,11 @@ class RoutedExperts(FeedForward):
         if s.score == "softmax_all":
             ops.moe_route_grouped(logits, s.top, ids, wts, experts=outputs, correction=self.correction, scale=s.route_scale,
                                   score="softmax", real=s.experts, groups=s.groups, keep=s.keep_groups,
-                                  group_top=s.group_top, renorm=s.renorm, renorm_eps=s.renorm_eps)
+                                  group_top=s.group_top, renorm=s.renorm, renorm_eps=s.renorm_eps, squared=s.weight_on == "input")
         elif s.score == "sigmoid":
             ops.moe_route_grouped(logits, s.top, ids, wts, experts=s.experts, correction=self.correction, groups=s.groups,
                                   keep=s.keep_groups, group_top=s.group_top, scale=s.route_scale, renorm=s.renorm,
-                                  renorm_eps=s.renorm_eps)
+                                  renorm_eps=s.renorm_eps, squared=s.weight_on == "input")
         else:
             ops.moe_route(logits, s.top, ids, wts, experts=s.experts, scale=s.route_scale)
         out = ws.get("ffn_out", (T, s.hidden), rt.act_dtype)

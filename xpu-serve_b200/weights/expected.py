@@ -1,6 +1,7 @@
 """The tensors a model spec expects, by full name, from its parts' declarations."""
 from __future__ import annotations
 
+from dataclasses import replace
 from typing import Dict, Optional, Sequence
 
 from ..config.spec import ModelSpec
@@ -35,6 +36,8 @@ def expected_tensors(spec: ModelSpec, prefix: Optional[str] = None) -> Dict[str,
         out[p + name] = TensorSpec(tuple(shape))
     for layer in spec.layers:
         for rel, ts in layer_tensors(layer).items():
+            if ts.free:       # (labels are a layer's own)
+                ts = replace(ts, free=tuple((axis, layer.prefix + label) for axis, label in ts.free))
             out[p + layer.prefix + rel] = ts
     return out
 

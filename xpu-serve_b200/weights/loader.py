@@ -43,8 +43,17 @@ def check_store(spec: ModelSpec, store: WeightStore) -> str:
     unexpected = [n for n in store.names() if n not in expected
                   and (not wrapped or n.startswith(prefix) or n == spec.names["head"])
                   and not any(pat.search(n) for pat in ignorable)]
-    wrong = [f"{n} is {list(store.shape(n))}, expected {list(ts.shape)}"
-             for n, ts in expected.items() if n in store and tuple(store.shape(n)) != tuple(ts.shape)]
+    free: Dict[str, int] = {}          # sizes that the checkpoint decides, by label: the first tensor's counts for the others
+    wrong = []
+    for n, ts in expected.items():
+        if n not in store:
+            continue
+        have, want = tuple(store.shape(n)), list(ts.shape)
+        for axis, label in ts.free:
+            if axis < len(have) and have[axis] > 0:
+                want[axis] = free.setdefault(label, have[axis])
+        if have != tuple(want):
+            wrong.append(f"{n} is {list(have)}, expected {want}")
     bad_dtype = [f"{n} is {store.dtype(n)}" for n in expected
                  if n in store and not (store.dtype(n).is_floating_point or
                                         store.dtype(n) in (torch.int32, torch.int64, torch.int16, torch.int8,
