@@ -276,6 +276,54 @@ def run_gararax_stacks(batch: int, steps: int, warmup: int, only=None) -> int:
     return run_stacks("gararax", GARARAX_STACKS, gararax_stack_configs, batch, steps, warmup, only)
 
 
+# Lazovik layer stacks (`--workload lazovik`; random weights), each beside the closest existing stack of equal width, layer count
+# and vocabulary: gated linear attention beside Vekuzen's memory with a constant decay per head, at the same head sizes; block
+# attention (filtered projections, capped scores) summed with time mixing, beside Tozarax's windowed attention of the same heads
+# summed with the gated delta rule over a state of the same size; all with routed experts. The first stack starts with the vector
+# that a pass over repeated layers starts with. `gla_wide` has fewer, larger memories.
+_L_MOE = {"kind": "moe", "expert": {"ff": 1024}, "router": {"experts": 16, "top": 4}, "shared": {"ff": 1024}}
+
+
+def _gla(heads, dim, vdim):
+    return "gla", {"heads": heads, "dim": dim, "vdim": vdim, "tau": 16.0, "rank": 64}
+
+
+LAZOVIK_STACKS = {
+    "gla_experts": (([(*_gla(16, 64, 128), _L_MOE)] * 2, {"start": 0, "stop": 2, "times": 1}), ("vekuzen", "lightning_experts")),
+    "gla_wide": (([(*_gla(8, 128, 256), None)] * 2, None),
+                 ("vekuzen", [("lightning", {"heads": 8, "dim": 128, "vdim": 256, "decay": [1.0 - 2.0 ** -(2 + h) for h in range(8)]}, None)] * 2)),
+    "parallel_experts": (([("parallel", {
+        "left": {"heads": 32, "kv_heads": 8, "dim": 64, "vdim": 64, "conv": 4, "mask": {"size": 1024}, "scale": 0.125, "softcap": 50.0,
+                 "rot": {"base": 500000.0, "dims": 32, "scaling": {"factor": 4.0, "original": 4096, "fast": 32.0, "slow": 1.0}}},
+        "right": {"heads": 32, "dim": 64, "rank": 64}, "left_scale": 0.7, "right_scale": 0.7}, _L_MOE)] * 2, None),
+        ("tozarax", [(_blocked(32, 8, 64, 64, 1024), _delta(16, 16, 64, 128), _T_MOE)] * 2)),
+}
+
+
+def lazovik_stack_configs(name: str, width: int = 2048, vocab: int = 32768):
+    from xpu_serve_b200.config import LazovikConfig, TozaraxConfig, VekuzenConfig
+    (layers, loop), (label, beside) = LAZOVIK_STACKS[name]
+    ours = {"architecture": "Lazovik", "width": width, "vocab": vocab, "norm": {"eps": 1e-5},
+            "layers": [{"type": t, "mixer": m, "mlp": f} for t, m, f in layers]}
+    if loop:
+        ours["loop"] = loop
+    ours = LazovikConfig.from_json(ours)
+    if isinstance(beside, str):
+        return ours, (label, vekuzen_stack_configs(beside, width, vocab)[0])
+    if label == "vekuzen":
+        other = {"architecture": "Vekuzen", "width": width, "vocab": vocab, "max_positions": CONTEXT, "norm": {"eps": 1e-6},
+                 "embedding": {"scale": 1.0}, "logit_scale": 0.5, "token_side": {"dim": 256},
+                 "layers": [{"type": t, "mixer": m, "mlp": f} for t, m, f in beside]}
+        return ours, (label, VekuzenConfig.from_json(other))
+    other = {"architecture": "Tozarax", "width": width, "vocab": vocab, "max_positions": CONTEXT, "norm": {"eps": 1e-5}, "canon": {"taps": 4},
+             "layers": [{"type": "parallel", "mixer": {"left": l, "right": r}, "mlp": f} for l, r, f in beside]}
+    return ours, (label, TozaraxConfig.from_json(other))
+
+
+def run_lazovik_stacks(batch: int, steps: int, warmup: int, only=None) -> int:
+    return run_stacks("lazovik", LAZOVIK_STACKS, lazovik_stack_configs, batch, steps, warmup, only)
+
+
 def run_stacks(workload: str, stacks, configs_of, batch: int, steps: int, warmup: int, only=None) -> int:
     """Prefill (one prompt of 2,048 tokens in one step) and decode (batch 8 after 2,048-token prompts, CUDA graph) of
     each stack of the workload and of the stack beside it, device-timed as the headline's points are. With XS_PROFILE=1
@@ -642,8 +690,8 @@ def main() -> int:
                          "at long context), which the default run adds to `points`")
     ap.add_argument("--only", default=None, choices=["decode", "prefill", "sample"],
                     help="time one part only and print a short line (for profiler captures)")
-    ap.add_argument("--stacks", default=None, help="with --workload saralix, nimelorn, tozarax, vekuzen or gararax: a comma list of the stacks to run (all)")
-    ap.add_argument("--workload", default=None, choices=sorted(WORKLOADS) + ["saralix", "nimelorn", "tozarax", "vekuzen", "gararax"],
+    ap.add_argument("--stacks", default=None, help="with --workload saralix, nimelorn, tozarax, vekuzen, gararax or lazovik: a comma list of the stacks to run (all)")
+    ap.add_argument("--workload", default=None, choices=sorted(WORKLOADS) + ["saralix", "nimelorn", "tozarax", "vekuzen", "gararax", "lazovik"],
                     help="instead of the default run: a batch of unequal prompts at another shape of the family")
     args = ap.parse_args()
 
@@ -661,6 +709,8 @@ def main() -> int:
         return run_saralix_stacks(args.batch or 8, args.steps or 128, args.warmup, args.stacks.split(",") if args.stacks else None)
     if args.workload == "nimelorn":
         return run_nimelorn_stacks(args.batch or 8, args.steps or 128, args.warmup, args.stacks.split(",") if args.stacks else None)
+    if args.workload == "lazovik":
+        return run_lazovik_stacks(args.batch or 8, args.steps or 128, args.warmup, args.stacks.split(",") if args.stacks else None)
     if args.workload == "gararax":
         return run_gararax_stacks(args.batch or 8, args.steps or 128, args.warmup, args.stacks.split(",") if args.stacks else None)
     if args.workload == "vekuzen":

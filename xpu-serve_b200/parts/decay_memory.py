@@ -56,7 +56,7 @@ class DecayMemoryMixer(Mixer):
         self.chunk = int(os.environ["XS_DECAY_CHUNK"]) if "XS_DECAY_CHUNK" in os.environ else None
 
     def scale_output(self, s: float) -> bool:
-        self.w_norm *= s
+        self.w_norm = self.w_norm * s
         return True
 
     def forward(self, x, step, cache, into=None) -> Optional[torch.Tensor]:
