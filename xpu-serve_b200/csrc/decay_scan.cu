@@ -49,6 +49,12 @@ int scan(const DecayScanArgs& a, int items, int dtype, cudaStream_t stream) {
 // 1 when xs_decay_scan finishes a head's output itself (norm, weight, gate).
 XS_API int xs_decay_scan_finishes(int D, int E) { return E <= 32 * columns_per_lane(D, E) ? 1 : 0; }
 
+// CTAs that run at one time on an SM, by the registers they are bounded for.
+XS_API int xs_decay_scan_ctas(int D, int E) {
+    const int cpl = columns_per_lane(D, E);
+    return D <= 32 ? scan_ctas(8, 4, cpl) : D <= 64 ? scan_ctas(16, 4, cpl) : D <= 128 ? scan_ctas(16, 8, cpl) : scan_ctas(32, 8, cpl);
+}
+
 // CTAs of one (sequence or chunk).
 XS_API int xs_decay_scan_blocks(int H, int D, int E) { return H * ceil_div_i(E, 32 * columns_per_lane(D, E)); }
 

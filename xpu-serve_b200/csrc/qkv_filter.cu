@@ -182,12 +182,171 @@ __global__ void qkv_filter_kernel(const QkvFilterArgs a) {
     }
 }
 
+// The same for long steps, kTile tokens a block: a channel's taps, bias and norm weights and the rows that neighbouring tokens
+// share are read once for all of them. Only what a sequence's first TAPS - 1 tokens of the step look back to comes from its state.
+constexpr int kTile = 4;
+
+template <typename T, int TAPS>
+__global__ void __launch_bounds__(256, 3) qkv_filter_tile_kernel(const QkvFilterArgs a, int n_tokens) {
+    constexpr int V = 4, ROWS = kTile + TAPS - 1;
+    extern __shared__ __align__(16) float f_sm[];        // [kTile][q and k channels]
+    __shared__ float red[2 * kTile][16];
+    pdl_launch_dependents();
+    const int t0 = blockIdx.x * kTile;
+    const int nq = a.Hq * a.D, nk = a.Hkv * a.D, C = nq + nk + a.Hkv * a.DV;
+    int pos[kTile], local[kTile], seq[kTile];
+    T* kpage[kTile];
+#pragma unroll
+    for (int i = 0; i < kTile; ++i) {
+        const int t = min(t0 + i, n_tokens - 1);
+        seq[i] = a.seq_of_token[t];
+        pos[i] = a.positions[t];
+    }
+#pragma unroll
+    for (int i = 0; i < kTile; ++i) {
+        local[i] = min(t0 + i, n_tokens - 1) - a.cu_seqlens[seq[i]];
+        const int page = a.page_table[(int64_t)seq[i] * a.P + pos[i] / a.page_size];
+        kpage[i] = (T*)a.pool + (int64_t)page * a.Hkv * a.page_size * (a.D + a.DV);
+    }
+    const T* x = (const T*)a.x;
+    pdl_wait();
+    float ssq[kTile], ssk[kTile];
+#pragma unroll
+    for (int i = 0; i < kTile; ++i) ssq[i] = ssk[i] = 0.0f;
+    for (int c = threadIdx.x * V; c < C; c += blockDim.x * V) {
+        float rows[ROWS][V], w[TAPS][V], bias[V];
+#pragma unroll
+        for (int r = 0; r < ROWS; ++r) {                  // row r is token t0 - (TAPS - 1) + r
+            const int t = t0 - (TAPS - 1) + r;
+#pragma unroll
+            for (int v = 0; v < V; ++v) rows[r][v] = 0.0f;
+            if (t >= 0 && t < n_tokens) Chans<T, V>::load(x + (int64_t)t * a.ld + c, rows[r]);
+        }
+#pragma unroll
+        for (int b = 0; b < TAPS; ++b) Chans<float, V>::load(a.taps + (int64_t)b * C + c, w[b]);
+#pragma unroll
+        for (int v = 0; v < V; ++v) bias[v] = 0.0f;
+        if (a.bias != nullptr) Chans<float, V>::load(a.bias + c, bias);
+#pragma unroll
+        for (int i = 0; i < kTile; ++i) {
+            if (t0 + i >= n_tokens) break;
+            float f[V];
+#pragma unroll
+            for (int v = 0; v < V; ++v) f[v] = 0.0f;
+#pragma unroll
+            for (int b = TAPS - 1; b >= 0; --b) {
+                if (pos[i] - b < 0) continue;             // before the sequence: zeros
+                if (local[i] - b >= 0) {
+#pragma unroll
+                    for (int v = 0; v < V; ++v) f[v] = fmaf(w[b][v], rows[i + TAPS - 1 - b][v] + bias[v], f[v]);
+                } else {
+                    float sv[V];
+                    Chans<T, V>::load((const T*)a.state + ((int64_t)a.slots[seq[i]] * (TAPS - 1) + (TAPS - 1 - (b - local[i]))) * C + c, sv);
+#pragma unroll
+                    for (int v = 0; v < V; ++v) f[v] = fmaf(w[b][v], sv[v] + bias[v], f[v]);
+                }
+            }
+            if (c < nq + nk) {
+                float ss = 0.0f;
+#pragma unroll
+                for (int v = 0; v < V; ++v) ss = fmaf(f[v], f[v], ss);
+                if (c < nq) ssq[i] += ss;
+                else ssk[i] += ss;
+                Chans<float, V>::store(f_sm + i * (nq + nk) + c, f);
+            } else {
+                const int vc = c - nq - nk, vh = vc / a.DV;
+                Chans<T, V>::store(kpage[i] + (int64_t)a.Hkv * a.page_size * a.D + ((int64_t)vh * a.page_size + pos[i] % a.page_size) * a.DV + (vc - vh * a.DV), f);
+            }
+        }
+    }
+    {
+        const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, warps = (blockDim.x + 31) >> 5;
+#pragma unroll
+        for (int i = 0; i < kTile; ++i) {
+            ssq[i] = warp_sum(ssq[i]);
+            ssk[i] = warp_sum(ssk[i]);
+            if (lane == 0) {
+                red[2 * i][warp] = ssq[i];
+                red[2 * i + 1][warp] = ssk[i];
+            }
+        }
+        __syncthreads();                                  // (the filtered values are in shared memory too)
+#pragma unroll
+        for (int i = 0; i < kTile; ++i) {
+            ssq[i] = warp_sum(lane < warps ? red[2 * i][lane] : 0.0f);
+            ssk[i] = warp_sum(lane < warps ? red[2 * i + 1][lane] : 0.0f);
+        }
+    }
+    const int half = a.D >> 1, pairs = (nq + nk) >> 1;
+    for (int e = threadIdx.x * V; e < pairs; e += blockDim.x * V) {
+        const int h = e / half, p = e - h * half;
+        const int lo = h * a.D + p, hi = lo + half;
+        const bool is_q = h < a.Hq;
+        const float* wt = is_q ? a.q_w : a.k_w;
+        float wu[V], wv[V];
+#pragma unroll
+        for (int v = 0; v < V; ++v) wu[v] = wv[v] = 1.0f;
+        if (wt != nullptr) {
+            Chans<float, V>::load(wt + (is_q ? lo : lo - nq), wu);
+            Chans<float, V>::load(wt + (is_q ? hi : hi - nq), wv);
+        }
+#pragma unroll
+        for (int i = 0; i < kTile; ++i) {
+            if (t0 + i >= n_tokens) break;
+            float y[V], z[V];
+            Chans<float, V>::load(f_sm + i * (nq + nk) + lo, y);
+            Chans<float, V>::load(f_sm + i * (nq + nk) + hi, z);
+            if (wt != nullptr) {
+                const float inv = is_q ? 1.0f / sqrtf(ssq[i] / a.q_count + a.eps) : 1.0f / sqrtf(ssk[i] / a.k_count + a.eps);
+#pragma unroll
+                for (int v = 0; v < V; ++v) {
+                    y[v] = y[v] * inv * wu[v];
+                    z[v] = z[v] * inv * wv[v];
+                }
+            }
+            if (a.rope != nullptr) {
+                const float4* cs = reinterpret_cast<const float4*>(a.rope + (int64_t)pos[i] * half + p);
+                const float4 c0 = cs[0], c1 = cs[1];
+                const float co[V] = {c0.x, c0.z, c1.x, c1.z}, si[V] = {c0.y, c0.w, c1.y, c1.w};
+#pragma unroll
+                for (int v = 0; v < V; ++v) {
+                    const float a0 = y[v] * co[v] - z[v] * si[v], a1 = z[v] * co[v] + y[v] * si[v];
+                    y[v] = a0;
+                    z[v] = a1;
+                }
+            }
+            T* dst = is_q ? (T*)a.q_out + (int64_t)(t0 + i) * nq + lo : kpage[i] + ((int64_t)(h - a.Hq) * a.page_size + pos[i] % a.page_size) * a.D + p;
+            Chans<T, V>::store(dst, y);
+            Chans<T, V>::store(dst + half, z);
+        }
+    }
+}
+
+template <typename T, int TAPS>
+void launch_tile(const QkvFilterArgs& a, int Tn, cudaStream_t stream) {
+    const int groups = ceil_div_i(a.Hq * a.D + a.Hkv * (a.D + a.DV), 4);
+    const int rounds = ceil_div_i(groups, 256);
+    const int threads = ceil_div_i(ceil_div_i(groups, rounds), 32) * 32;      // every thread the same number of channels, but for the last warp's
+    const size_t smem = (size_t)kTile * (a.Hq + a.Hkv) * a.D * sizeof(float);
+    if (smem > 40 * 1024)
+        cudaFuncSetAttribute(qkv_filter_tile_kernel<T, TAPS>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    xs_launch(qkv_filter_tile_kernel<T, TAPS>, dim3(ceil_div_i(Tn, kTile)), dim3(threads), smem, stream, a, Tn);
+}
+
 template <typename T>
 int launch_filter(const QkvFilterArgs& a, int Tn, bool vec, cudaStream_t stream) {
     const int C = a.Hq * a.D + a.Hkv * (a.D + a.DV);
     const size_t smem = (size_t)(a.Hq + a.Hkv) * a.D * sizeof(float);
     const int work = vec ? ceil_div_i(C, 4) : C;
     const int threads = work >= 512 ? 512 : work >= 256 ? 256 : 128;
+    if (vec && !a.move_state && Tn >= 256 && a.n <= 5 && smem * kTile <= 160 * 1024 && (uintptr_t)a.rope % 16 == 0) {
+        if (a.n == 1) launch_tile<T, 1>(a, Tn, stream);
+        else if (a.n == 2) launch_tile<T, 2>(a, Tn, stream);
+        else if (a.n == 3) launch_tile<T, 3>(a, Tn, stream);
+        else if (a.n == 4) launch_tile<T, 4>(a, Tn, stream);
+        else launch_tile<T, 5>(a, Tn, stream);
+        return 0;
+    }
 #define XS_GO2(V, N)                                                                                                       \
     do {                                                                                                                   \
         if (smem > 47 * 1024)                                                                                              \

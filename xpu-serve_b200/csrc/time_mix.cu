@@ -78,65 +78,100 @@ __global__ void token_mix_vec_kernel(const __nv_bfloat16* __restrict__ x, int64_
 
 enum DecayKind : int { kDoubleExp = 0, kRootedSigmoid = 1 };
 
+// FAST (beside weights of 8 bits of mantissa): the hardware's exponential and logarithm, a few units in the last place of
+// float32; float32 weights take the exact functions.
+template <bool FAST>
 __device__ __forceinline__ float decay_of(float v, int kind, float power) {
-    if (kind == kDoubleExp) return expf(-expf(v));
+    if (kind == kDoubleExp) return FAST ? __expf(-__expf(v)) : expf(-expf(v));
     // sigmoid(v)^power = exp(power * log sigmoid(v)), log sigmoid(v) = min(v, 0) - log(1 + exp(-|v|))
-    return expf(power * (fminf(v, 0.0f) - log1pf(expf(-fabsf(v)))));
+    if constexpr (FAST) return __expf(power * (fminf(v, 0.0f) - __logf(1.0f + __expf(-fabsf(v)))));
+    else return expf(power * (fminf(v, 0.0f) - log1pf(expf(-fabsf(v)))));
 }
 
-constexpr int kRankStep = 32;    // hidden entries staged at a time
+constexpr int kRankStep = 64;    // hidden entries staged at a time
+constexpr int kDecayCols = 64;   // channels a block: a lane has two of them
 
-// 4 warps: a lane is a channel of 32, a warp TPW tokens.
+// 4 warps: a lane is two channels, a warp TPW tokens at a time; a block walks `tiles` tiles of 4 TPW tokens with its channels'
+// weights staged once (where the rank is at most kRankStep). wvec: rows of w may be read 16 bytes at a time.
 template <typename TW, int TPW>
 __global__ void __launch_bounds__(128) low_rank_decay_kernel(const float* __restrict__ z, int64_t ldz, const TW* __restrict__ w,
                                                              const float* __restrict__ bias, float* __restrict__ out, int Tn, int C, int R,
-                                                             int hidden_tanh, int kind, float power) {
-    __shared__ float ws[kRankStep][33];
+                                                             int hidden_tanh, int kind, float power, int tiles, int wvec) {
+    __shared__ float ws[kRankStep][kDecayCols + 1];
     __shared__ __align__(16) float zs[4 * TPW][kRankStep];
     pdl_launch_dependents();
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
-    const int c0 = blockIdx.x * 32, t0 = blockIdx.y * (4 * TPW);
-    float acc[TPW];
-#pragma unroll
-    for (int i = 0; i < TPW; ++i) acc[i] = 0.0f;
-    const float b = bias != nullptr && c0 + lane < C ? bias[c0 + lane] : 0.0f;
+    const int c0 = blockIdx.x * kDecayCols;
+    const float b0 = bias != nullptr && c0 + lane < C ? bias[c0 + lane] : 0.0f;
+    const float b1 = bias != nullptr && c0 + lane + 32 < C ? bias[c0 + lane + 32] : 0.0f;
     bool waited = false;
-    for (int r0 = 0; r0 < R; r0 += kRankStep) {
-        __syncthreads();
-        for (int e = threadIdx.x; e < 32 * kRankStep; e += 128) {
-            const int c = e >> 5, r = e & 31;
-            ws[r][c] = c0 + c < C && r0 + r < R ? to_f32(w[(int64_t)(c0 + c) * R + r0 + r]) : 0.0f;
-        }
-        if (!waited) {                             // (the weights depend on nothing)
-            pdl_wait();
-            waited = true;
-        }
-        for (int e = threadIdx.x; e < 4 * TPW * kRankStep; e += 128) {
-            const int t = e >> 5, r = e & 31;
-            float v = t0 + t < Tn && r0 + r < R ? z[(int64_t)(t0 + t) * ldz + r0 + r] : 0.0f;
-            if (hidden_tanh) v = tanhf(v);
-            zs[t][r] = v;
-        }
-        __syncthreads();
+    for (int tile = 0; tile < tiles; ++tile) {
+        const int t0 = (blockIdx.y * tiles + tile) * (4 * TPW);
+        if (t0 >= Tn) break;
+        float acc[TPW][2];
 #pragma unroll
-        for (int r = 0; r < kRankStep; r += 4) {
-            const float w0 = ws[r][lane], w1 = ws[r + 1][lane], w2 = ws[r + 2][lane], w3 = ws[r + 3][lane];
+        for (int i = 0; i < TPW; ++i) acc[i][0] = acc[i][1] = 0.0f;
+        for (int r0 = 0; r0 < R; r0 += kRankStep) {
+            __syncthreads();
+            if (tile == 0 || R > kRankStep) {
+                if (wvec) {
+                    constexpr int N = 16 / sizeof(TW);
 #pragma unroll
-            for (int i = 0; i < TPW; ++i) {
-                const float4 v = *reinterpret_cast<const float4*>(&zs[warp * TPW + i][r]);
-                acc[i] = fmaf(w0, v.x, acc[i]);
-                acc[i] = fmaf(w1, v.y, acc[i]);
-                acc[i] = fmaf(w2, v.z, acc[i]);
-                acc[i] = fmaf(w3, v.w, acc[i]);
+                    for (int e = threadIdx.x; e < kDecayCols * kRankStep / N; e += 128) {
+                        const int c = e / (kRankStep / N), r = (e - c * (kRankStep / N)) * N;
+                        uint4 raw = make_uint4(0u, 0u, 0u, 0u);
+                        if (c0 + c < C && r0 + r < R) raw = *reinterpret_cast<const uint4*>(w + (int64_t)(c0 + c) * R + r0 + r);
+                        const TW* v = reinterpret_cast<const TW*>(&raw);
+#pragma unroll
+                        for (int j = 0; j < N; ++j) ws[r + j][c] = to_f32(v[j]);
+                    }
+                } else {
+                    for (int e = threadIdx.x; e < kDecayCols * kRankStep; e += 128) {
+                        const int c = e / kRankStep, r = e - c * kRankStep;
+                        ws[r][c] = c0 + c < C && r0 + r < R ? to_f32(w[(int64_t)(c0 + c) * R + r0 + r]) : 0.0f;
+                    }
+                }
+            }
+            if (!waited) {                             // (the weights depend on nothing)
+                pdl_wait();
+                waited = true;
+            }
+#pragma unroll 4
+            for (int e = threadIdx.x; e < 4 * TPW * kRankStep; e += 128) {
+                const int t = e / kRankStep, r = e - t * kRankStep;
+                float v = t0 + t < Tn && r0 + r < R ? z[(int64_t)(t0 + t) * ldz + r0 + r] : 0.0f;
+                if (hidden_tanh) v = tanhf(v);
+                zs[t][r] = v;
+            }
+            __syncthreads();
+            const int steps = min(kRankStep, R - r0);      // (entries from R on are zero: whole fours)
+            for (int r = 0; r < steps; r += 4) {
+                float u[4][2];
+#pragma unroll
+                for (int j = 0; j < 4; ++j) {
+                    u[j][0] = ws[r + j][lane];
+                    u[j][1] = ws[r + j][lane + 32];
+                }
+#pragma unroll
+                for (int i = 0; i < TPW; ++i) {
+                    const float4 v = *reinterpret_cast<const float4*>(&zs[warp * TPW + i][r]);
+                    const float vv[4] = {v.x, v.y, v.z, v.w};
+#pragma unroll
+                    for (int j = 0; j < 4; ++j) {
+                        acc[i][0] = fmaf(u[j][0], vv[j], acc[i][0]);
+                        acc[i][1] = fmaf(u[j][1], vv[j], acc[i][1]);
+                    }
+                }
             }
         }
-    }
-    const int c = c0 + lane;
-    if (c >= C) return;
+        const int c = c0 + lane;
 #pragma unroll
-    for (int i = 0; i < TPW; ++i) {
-        const int t = t0 + warp * TPW + i;
-        if (t < Tn) out[(int64_t)t * C + c] = decay_of(acc[i] + b, kind, power);
+        for (int i = 0; i < TPW; ++i) {
+            const int t = t0 + warp * TPW + i;
+            if (t >= Tn) break;
+            if (c < C) out[(int64_t)t * C + c] = decay_of<sizeof(TW) == 2>(acc[i][0] + b0, kind, power);
+            if (c + 32 < C) out[(int64_t)t * C + c + 32] = decay_of<sizeof(TW) == 2>(acc[i][1] + b1, kind, power);
+        }
     }
 }
 
@@ -170,14 +205,19 @@ XS_API int xs_low_rank_decay(const float* z, int64_t ldz, const void* w, int w_d
     XS_REQUIRE(T > 0 && C > 0 && R > 0 && ldz >= R && (kind == kDoubleExp || kind == kRootedSigmoid) && power > 0.0f,
                "low_rank_decay: %d tokens, %d channels, rank %d, kind %d", T, C, R, kind);
     XS_REQUIRE(T <= 65535 * 8, "low_rank_decay: %d tokens exceed the grid limit", T);
+    const int cols = ceil_div_i(C, kDecayCols);
+    const int wvec = (R * (w_dtype == XS_BF16 ? 2 : 4)) % 16 == 0 && (uintptr_t)w % 16 == 0;
     if (T >= 256) {
+        const int all = ceil_div_i(T, 32);
+        int tiles = ceil_div_i((int64_t)all * cols, 148 * 8);          // about one round of blocks
+        if (tiles > 8) tiles = 8;
         XS_DISPATCH_DTYPE(w_dtype, TW,
-                          xs_launch(low_rank_decay_kernel<TW, 8>, dim3(ceil_div_i(C, 32), ceil_div_i(T, 32)), dim3(128), 0, stream, z, ldz,
-                                    (const TW*)w, bias, out, T, C, R, hidden_tanh, kind, power));
+                          xs_launch(low_rank_decay_kernel<TW, 8>, dim3(cols, ceil_div_i(all, tiles)), dim3(128), 0, stream, z, ldz,
+                                    (const TW*)w, bias, out, T, C, R, hidden_tanh, kind, power, tiles, wvec));
     } else {
         XS_DISPATCH_DTYPE(w_dtype, TW,
-                          xs_launch(low_rank_decay_kernel<TW, 2>, dim3(ceil_div_i(C, 32), ceil_div_i(T, 8)), dim3(128), 0, stream, z, ldz,
-                                    (const TW*)w, bias, out, T, C, R, hidden_tanh, kind, power));
+                          xs_launch(low_rank_decay_kernel<TW, 2>, dim3(cols, ceil_div_i(T, 8)), dim3(128), 0, stream, z, ldz,
+                                    (const TW*)w, bias, out, T, C, R, hidden_tanh, kind, power, 1, wvec));
     }
     XS_LAUNCH_CHECK("low_rank_decay");
     return 0;

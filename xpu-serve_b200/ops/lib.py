@@ -102,7 +102,7 @@ def _signatures(lib) -> None:
         fn.restype = c_int
     lib.xs_last_error.restype = ctypes.c_char_p
     lib.xs_last_error.argtypes = []
-    for name, args in (("xs_decay_scan_finishes", [c_int, c_int]), ("xs_decay_scan_blocks", [c_int, c_int, c_int])):
+    for name, args in (("xs_decay_scan_finishes", [c_int, c_int]), ("xs_decay_scan_ctas", [c_int, c_int]), ("xs_decay_scan_blocks", [c_int, c_int, c_int])):
         getattr(lib, name).restype, getattr(lib, name).argtypes = c_int, args
     lib.xs_uniform.restype = c_double
     lib.xs_uniform.argtypes = [c_uint64, c_uint64]
@@ -1591,6 +1591,11 @@ def low_rank_decay(z: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor
 def decay_scan_finishes(dim: int, vdim: int) -> bool:
     """Whether decay_scan can norm and gate the heads' outputs itself."""
     return bool(load().xs_decay_scan_finishes(dim, vdim))
+
+
+def decay_scan_ctas(dim: int, vdim: int) -> int:
+    """CTAs of the scan that run at one time on an SM."""
+    return int(load().xs_decay_scan_ctas(dim, vdim))
 
 
 def decay_scan_blocks(heads: int, dim: int, vdim: int) -> int:

@@ -52,7 +52,7 @@ class DecayMemoryMixer(Mixer):
         self.b_o = None
         self.finishes = ops.decay_scan_finishes(spec.dim, vdim)
         # Pieces of at least two chunks run chunk by chunk side by side. XS_DECAY_CHUNK: tokens a chunk (0: always in order);
-        # unset: as many chunks as fill the device once with four CTAs an SM, between 32 and 256 tokens each.
+        # unset: as many chunks as fill the device once, between 32 and 256 tokens each.
         self.chunk = int(os.environ["XS_DECAY_CHUNK"]) if "XS_DECAY_CHUNK" in os.environ else None
 
     def scale_output(self, s: float) -> bool:
@@ -75,7 +75,7 @@ class DecayMemoryMixer(Mixer):
         T = q.shape[0]
         chunk, chunks = self.chunk, None
         if chunk is None:
-            at_once = max(1, (4 * rt.sm_count) // ops.decay_scan_blocks(s.heads, s.dim, self.vdim))
+            at_once = max(1, (ops.decay_scan_ctas(s.dim, self.vdim) * rt.sm_count) // ops.decay_scan_blocks(s.heads, s.dim, self.vdim))
             chunk = min(256, max(32, -(-T // at_once // 8) * 8))
         if chunk > 0 and not step.fixed_shape and not step.decode and step.max_q_len >= 2 * chunk:
             chunk_seq, first_chunk = chunk_plan(step, chunk, rt.device)
